@@ -139,7 +139,7 @@ NXD_DEVICE uint32_t mapa_shared(uint32_t addr, uint32_t cta) {
 }
 NXD_DEVICE void mbar_arrive_cluster(uint32_t cluster_addr) {
   // default semantics (.release at CTA scope) as in cutlass::arch::ClusterBarrier::arrive(cta_id): a cluster-scope
-  // release would compile to MEMBAR.ALL.GPU + ERRBAR on every arrive (measured: 3x slower producer loop)
+  // release on every arrive made the producer loop 3x slower (timed)
   asm volatile("mbarrier.arrive.shared::cluster.b64 _, [%0];" ::"r"(cluster_addr) : "memory");
 }
 constexpr uint32_t kPeerBitMask = 0xFEFFFFFFu;   // clears the CTA-rank bit of a shared::cluster address → leader CTA
@@ -171,7 +171,7 @@ NXD_DEVICE void tcgen05_mma_f16_2cta(uint32_t tmem_d, uint64_t desc_a, uint64_t 
 
 
 // ---- elected issue: the whole (converged) MMA warp executes these; one elected lane runs the tcgen05 instruction.
-// Issuing from `if (lane == 0)` makes nvcc wrap every MMA issue in an election loop (~100 cycles per MMA, measured).  For the attention kernels (32-64-cycle UMMAs) that made the issuing thread the
+// Issuing from `if (lane == 0)` costs ~100 cycles per MMA (timed).  For the attention kernels (32-64-cycle UMMAs) that made the issuing thread the
 // bottleneck and the elected form fixed it.  For the big-tile GEMMs (128-cycle UMMAs) the elected form measured SLOWER
 // (8192^3: 1371 vs 1637 TFLOP/s — 32 lanes spinning on the mbarriers), so
 // the GEMM kernels keep single-lane issue; these helpers are kept for small-tile kernels.
