@@ -10,7 +10,9 @@
 //                  1: gelu_erf, 2: the matrix stacks gate rows over up rows and out = silu(gate row . x) * (up row . x), O/2 columns;
 //                  3: the square of relu; rows whose sel names no matrix give zeros
 //   moe_combine  : y[n,:] = base_weight[n] * base[n,:] + sum_k weight[n,k] * rows[src[n,k],:], summed in float
-//   route_topk   : scores, choice with a correction, top-k, weights and the identity experts' share in one launch
+//   route_topk   : scores, choice with a correction (optionally only among the best groups of neighbouring experts), top-k, weights
+//                  (optionally divided by their sum) and the identity experts' share or the shared expert's gate in one launch
+//   sigmoid_gate_heads : heads laid out [H, N, V] times sigmoid of a gate per coordinate, packed to [N, H * V]
 //   small_linear_f32 : a few rows times a matrix with float results (router logits, per-head scalars of the recurrences)
 #include "seq_common.cuh"
 #include "seqmix.h"
@@ -125,12 +127,17 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __rest
 // are chosen (ties: the lower index), in descending order; a chosen real expert (index < n_real) gets weight score * scale, a chosen
 // identity expert weight 0 while its score is added to ident[row].  Kind 2: the scores are the logits themselves and the weights
 // are the softmax over the CHOSEN logits only (times scale).  PL: logits per lane (E <= 32 PL).
+// groups > 0: the experts form `groups` equal runs of neighbours, a group is worth the sum of its two largest choice values, and only
+// experts of the `gkeep` best groups (ties: the lower index) can be chosen.  norm: the chosen scores are divided by their sum + 1e-20.
+// share: column E of the row is the logit of a gate, whose sigmoid goes to ident[row].
 template <int PL>
 __global__ void route_topk_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int N, int E, int top, int n_real,
-                                  int kind, float scale, float* __restrict__ w, long* __restrict__ idx, float* __restrict__ ident) {
+                                  int kind, float scale, int groups, int gkeep, int norm, int share, long z_stride, float* __restrict__ w,
+                                  long* __restrict__ idx, float* __restrict__ ident) {
+    __shared__ float room[4][32 * PL];
     const int row = blockIdx.x * blockDim.y + threadIdx.y, lane = threadIdx.x;
     if (row >= N) return;
-    const float* z = logits + (long)row * E;
+    const float* z = logits + (long)row * z_stride;
     float sc[PL], ch[PL];
     float mx = -INFINITY;
 #pragma unroll
@@ -157,6 +164,54 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, const float*
         const int e = lane + 32 * i;
         ch[i] = e < E ? sc[i] + (correction ? correction[e] : 0.f) : -INFINITY;
     }
+    if (groups > 0) {
+        float* mine = room[threadIdx.y];
+        const int n = E / groups;
+#pragma unroll
+        for (int i = 0; i < PL; ++i) mine[lane + 32 * i] = ch[i];
+        __syncwarp();
+        float worth[PL];
+#pragma unroll
+        for (int i = 0; i < PL; ++i) {
+            const int g = lane + 32 * i;
+            float a = -INFINITY, c = -INFINITY;                                  // the group's two largest
+            if (g < groups)
+                for (int e = g * n; e < (g + 1) * n; ++e) {
+                    const float v = mine[e];
+                    if (v > a) { c = a; a = v; } else c = fmaxf(c, v);
+                }
+            worth[i] = g < groups ? (n > 1 ? a + c : a) : -INFINITY;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < PL; ++i) mine[lane + 32 * i] = 0.f;                  // from here on: which groups stay
+        __syncwarp();
+        for (int t = 0; t < gkeep; ++t) {
+            float v = -INFINITY;
+            int g = 0x7fffffff;
+#pragma unroll
+            for (int i = 0; i < PL; ++i)
+                if (worth[i] > v) { v = worth[i]; g = lane + 32 * i; }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+                const int og = __shfl_xor_sync(0xffffffffu, g, o);
+                if (ov > v || (ov == v && og < g)) { v = ov; g = og; }
+            }
+            if (g < groups && (g & 31) == lane) {
+                mine[g] = 1.f;
+#pragma unroll
+                for (int i = 0; i < PL; ++i)
+                    if (lane + 32 * i == g) worth[i] = -INFINITY;
+            }
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < PL; ++i) {
+            const int e = lane + 32 * i;
+            if (e < E && mine[e / n] == 0.f) ch[i] = -INFINITY;
+        }
+    }
     float idw = 0.f, first = 0.f, total = 0.f, keep = 0.f;
     for (int t = 0; t < top; ++t) {
         float bv = -INFINITY, bs = 0.f;
@@ -178,36 +233,37 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, const float*
             for (int i = 0; i < PL; ++i)
                 if (lane + 32 * i == e) ch[i] = -INFINITY;
         }
-        if (kind == 2) {                                                         // every lane follows the sum; lane t keeps the t-th
+        if (kind == 2 || norm) {                                                 // every lane follows the sum; lane t keeps the t-th
             if (t == 0) first = s_e;                                             // exponential (the first chosen logit is the largest)
-            const float x = expf(s_e - first);
+            const float x = kind == 2 ? expf(s_e - first) : s_e;
             total += x;
             if (t == lane) keep = x;
             if (t >= 32 && lane == 0) w[(long)row * top + t] = x;                // beyond a warp's worth: through memory
         }
         if (lane == 0) {
             idx[(long)row * top + t] = e;
-            if (kind != 2) {
+            if (kind != 2 && !norm) {
                 w[(long)row * top + t] = e < n_real ? s_e * scale : 0.f;
                 if (e >= n_real) idw += s_e;
             }
         }
     }
-    if (kind == 2) {
+    if (kind == 2 || norm) {
+        if (norm) total += 1e-20f;
         if (lane < top) w[(long)row * top + lane] = keep / total * scale;
         if (top > 32 && lane == 0)
             for (int t = 32; t < top; ++t) w[(long)row * top + t] = w[(long)row * top + t] / total * scale;
     }
-    if (lane == 0 && ident) ident[row] = idw;
+    if (lane == 0 && ident) ident[row] = share ? sigmoidf_(z[E]) : idw;
 }
 
-bool route_topk(const float* logits, const float* correction, int N, int E, int top, int n_real, int kind, float scale, float* w, long* idx,
-                float* ident, cudaStream_t s) {
-    if (E > 256 || top > E) return false;
+bool route_topk(const float* logits, long z_stride, const float* correction, int N, int E, int top, int n_real, int kind, float scale, int groups,
+                int gkeep, int norm, int share, float* w, long* idx, float* ident, cudaStream_t s) {
+    if (E > 256 || top > E || (groups > 0 && (E % groups || gkeep < 1 || gkeep > groups || top > gkeep * (E / groups)))) return false;
     if (N == 0) return true;
     dim3 block(32, 4), grid((N + 3) / 4);
     const int pl = (E + 31) / 32;
-#define SEQMIX_ROUTE(P) route_topk_kernel<P><<<grid, block, 0, s>>>(logits, correction, N, E, top, n_real, kind, scale, w, idx, ident)
+#define SEQMIX_ROUTE(P) route_topk_kernel<P><<<grid, block, 0, s>>>(logits, correction, N, E, top, n_real, kind, scale, groups, gkeep, norm, share, z_stride, w, idx, ident)
     if (pl <= 1) SEQMIX_ROUTE(1); else if (pl <= 2) SEQMIX_ROUTE(2); else if (pl <= 4) SEQMIX_ROUTE(4); else SEQMIX_ROUTE(8);
 #undef SEQMIX_ROUTE
     return true;
@@ -362,6 +418,38 @@ void sigmoid_gate_mul(void* x, int bf, const void* gate, int gate_bf, long gate_
     else if (bf) sigmoid_gate_mul_kernel<bf16, float><<<blocks, 256, 0, s>>>((bf16*)x, (const float*)gate, gate_stride, rows, C, rep);
     else if (gate_bf) sigmoid_gate_mul_kernel<float, bf16><<<blocks, 256, 0, s>>>((float*)x, (const bf16*)gate, gate_stride, rows, C, rep);
     else sigmoid_gate_mul_kernel<float, float><<<blocks, 256, 0, s>>>((float*)x, (const float*)gate, gate_stride, rows, C, rep);
+}
+
+// ov [H, N, V] contiguous, gate [N, H * V] with its own row stride → out [N, H * V]: four coordinates per thread when V and the gate's
+// rows are in whole fours
+template <typename T, bool VEC>
+__global__ void sigmoid_gate_heads_kernel(const T* __restrict__ ov, const T* __restrict__ gate, long gate_stride, long N, int H, int V,
+                                          T* __restrict__ out) {
+    const long i = ((long)blockIdx.x * blockDim.x + threadIdx.x) * (VEC ? 4 : 1);
+    const int HV = H * V;
+    if (i >= N * HV) return;
+    const long n = i / HV;
+    const int c = (int)(i - n * HV), h = c / V, v = c - h * V;
+    const T* src = ov + ((long)h * N + n) * V + v;
+    const T* g = gate + n * gate_stride + c;
+    if (VEC) {
+        const float4 a = ld4(src), z = ld4(g);
+        st4(out + i, make_float4(a.x * sigmoidf_(z.x), a.y * sigmoidf_(z.y), a.z * sigmoidf_(z.z), a.w * sigmoidf_(z.w)));
+    } else {
+        stf(out + i, ldf(src) * sigmoidf_(ldf(g)));
+    }
+}
+
+void sigmoid_gate_heads(const void* ov, const void* gate, long gate_stride, int bf, long N, int H, int V, void* out, cudaStream_t s) {
+    const long total = N * H * V;
+    if (total == 0) return;
+    const size_t a4 = bf ? 8 : 16;
+    const bool vec = V % 4 == 0 && gate_stride % 4 == 0 && (uintptr_t)ov % a4 == 0 && (uintptr_t)gate % a4 == 0 && (uintptr_t)out % a4 == 0;
+    const unsigned blocks = (unsigned)((total / (vec ? 4 : 1) + 127) / 128);
+#define SEQMIX_SGH(T, V_) sigmoid_gate_heads_kernel<T, V_><<<blocks, 128, 0, s>>>((const T*)ov, (const T*)gate, gate_stride, N, H, V, (T*)out)
+    if (bf) { if (vec) SEQMIX_SGH(bf16, true); else SEQMIX_SGH(bf16, false); }
+    else { if (vec) SEQMIX_SGH(float, true); else SEQMIX_SGH(float, false); }
+#undef SEQMIX_SGH
 }
 
 void indexed_gemv(const void* w, const int* sel, const void* x, int bf, long x_stride, int M, int E, int O, int I, int act, void* out,

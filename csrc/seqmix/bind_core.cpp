@@ -17,11 +17,13 @@ Tensor short_conv(const Tensor& x, const Tensor& w, const c10::optional<Tensor>&
     return out;
 }
 
-// rows of x ([rows, C], row stride free) → out [rows, C] contiguous; w float [C] or one number
-Tensor rms_norm(const Tensor& x, const Tensor& w, double eps, const c10::optional<Tensor>& gate, bool out_bf16, bool center) {
+// rows of x ([rows, C], row stride free) → out [rows, C] contiguous; w float [C] or one number; bias float [C] or none
+Tensor rms_norm(const Tensor& x, const Tensor& w, double eps, const c10::optional<Tensor>& gate, bool out_bf16, bool center,
+                const c10::optional<Tensor>& bias) {
     TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.stride(1) == 1, "x must be [rows, C] with a contiguous last dimension");
     const int rows = x.size(0), C = x.size(1);
     TORCH_CHECK(w.numel() == 1 || w.numel() == C, "weight must hold 1 or C numbers");
+    TORCH_CHECK(!bias || bias->numel() == C, "bias must hold C numbers");
     Tensor out = at::empty({rows, C}, x.options().dtype(out_bf16 ? at::kBFloat16 : at::kFloat));
     const void* g = nullptr;
     long gs = 0;
@@ -32,7 +34,7 @@ Tensor rms_norm(const Tensor& x, const Tensor& w, double eps, const c10::optiona
     }
     if (rows)
         seqmix::rms_norm(x.data_ptr(), is_bf(x), x.stride(0), rows, C, f32(w), w.numel() == 1 ? 0 : 1, (float)eps, g, gs, out.data_ptr(),
-                         out_bf16, C, nullptr, 0, center, stream());
+                         out_bf16, C, nullptr, 0, center, bias ? f32(*bias) : nullptr, stream());
     check_launch();
     return out;
 }
@@ -45,7 +47,7 @@ void add_rms_norm_(Tensor res, const Tensor& y, const Tensor& w, double eps, boo
     TORCH_CHECK(res.size(0) == rows && res.size(1) == C && (w.numel() == 1 || w.numel() == C), "shape mismatch");
     if (rows)
         seqmix::rms_norm(y.data_ptr(), is_bf(y), y.stride(0), rows, C, f32(w), w.numel() == 1 ? 0 : 1, (float)eps, nullptr, 0, nullptr, 0, 0,
-                         res.data_ptr<float>(), res.stride(0), center, stream());
+                         res.data_ptr<float>(), res.stride(0), center, nullptr, stream());
     check_launch();
 }
 
@@ -162,6 +164,44 @@ void postnorm_gated_(Tensor x, const Tensor& y, const c10::optional<Tensor>& gat
     check_launch();
 }
 
+// x float [rows, C] (in place) += scale * y, then h = norm(x) * w + bias of y's dtype (undefined tensor without w).  y: [rows, C], or with
+// src / weight [rows, top] the contiguous expert rows [M, C] of a routed feed-forward (base [rows, C] times base_weight [rows] added).
+Tensor residual_norm_(Tensor x, const Tensor& y, const c10::optional<Tensor>& scale, const c10::optional<Tensor>& w,
+                      const c10::optional<Tensor>& bias, double eps, bool center, const c10::optional<Tensor>& src,
+                      const c10::optional<Tensor>& weight, const c10::optional<Tensor>& base, const c10::optional<Tensor>& base_weight) {
+    TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.stride(1) == 1 && x.scalar_type() == at::kFloat && y.dim() == 2 && y.stride(1) == 1 &&
+                    y.size(1) == x.size(1), "x must be float [rows, C], y rows of C numbers");
+    const int rows = x.size(0), C = x.size(1);
+    for (auto* t : {&scale, &w, &bias}) TORCH_CHECK(!*t || (*t)->numel() == C, "scale, weight and bias hold C numbers");
+    int top = 0;
+    if (src) {
+        TORCH_CHECK(weight && src->dim() == 2 && src->size(0) == rows && weight->sizes() == src->sizes() && y.is_contiguous(), "bad expert operands");
+        top = src->size(1);
+    } else {
+        TORCH_CHECK(y.size(0) == rows && !base, "one row of y per row of x");
+    }
+    if (base) TORCH_CHECK(base->is_contiguous() && base->scalar_type() == y.scalar_type() && base->size(0) == rows && base->size(1) == C, "bad base");
+    if (base_weight) TORCH_CHECK(base && base_weight->numel() == rows, "base_weight needs a base and one number per row");
+    Tensor h = w ? at::empty({rows, C}, y.options()) : Tensor();
+    seqmix::residual_norm(x.data_ptr<float>(), x.stride(0), y.data_ptr(), y.stride(0), is_bf(y), src ? i32(*src) : nullptr,
+                          weight ? f32(*weight) : nullptr, top, base ? base->data_ptr() : nullptr, base_weight ? f32(*base_weight) : nullptr,
+                          scale ? f32(*scale) : nullptr, w ? f32(*w) : nullptr, bias ? f32(*bias) : nullptr, (float)eps, center, rows, C,
+                          w ? h.data_ptr() : nullptr, C, stream());
+    check_launch();
+    return h;
+}
+
+// ov [H, N, V] contiguous, gate [N, H * V] of its dtype (row stride free) → [N, H * V] = heads packed, times sigmoid(gate)
+Tensor sigmoid_gate_heads(const Tensor& ov, const Tensor& gate) {
+    TORCH_CHECK(ov.is_cuda() && ov.dim() == 3 && ov.is_contiguous() && gate.dim() == 2 && gate.stride(1) == 1 && gate.size(0) == ov.size(1) &&
+                    gate.size(1) == ov.size(0) * ov.size(2) && gate.scalar_type() == ov.scalar_type(), "ov must be [H, N, V], gate [N, H * V]");
+    Tensor out = at::empty({ov.size(1), ov.size(0) * ov.size(2)}, ov.options());
+    seqmix::sigmoid_gate_heads(ov.data_ptr(), gate.data_ptr(), gate.stride(0), is_bf(ov), ov.size(1), (int)ov.size(0), (int)ov.size(2),
+                               out.data_ptr(), stream());
+    check_launch();
+    return out;
+}
+
 // x [rows, C], gate [rows, C] (row strides free), w float [C] or [C / groups] → out [rows, C] (row stride free) of the gate's dtype
 void group_rms_norm_gated(const Tensor& x, const Tensor& gate, const Tensor& w, int64_t groups, double eps, bool gate_first, Tensor out,
                           double out_scale, bool sigmoid_gate) {
@@ -175,17 +215,18 @@ void group_rms_norm_gated(const Tensor& x, const Tensor& gate, const Tensor& w, 
     check_launch();
 }
 
-// logits float [N,E] → (weights float [N,top], expert ids int64 [N,top], identity share float [N]); kind 1: softmax, 0: sigmoid
+// logits float [N,E] (one more column with `share`) → (weights float [N,top], expert ids int64 [N,top], identity share or gate float [N]);
+// kind 1: softmax, 0: sigmoid, 2: softmax over the chosen; groups / gkeep: the choice is limited to the best groups; norm: weights sum to 1
 std::vector<Tensor> route_topk(const Tensor& logits, const c10::optional<Tensor>& correction, int64_t top, int64_t n_real, int64_t kind,
-                               double scale) {
+                               double scale, int64_t groups, int64_t gkeep, bool norm, bool share) {
     TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.is_contiguous() && logits.scalar_type() == at::kFloat, "logits must be float [N,E]");
-    const int N = logits.size(0), E = logits.size(1);
+    const int N = logits.size(0), E = logits.size(1) - (share ? 1 : 0);
     TORCH_CHECK(!correction || correction->numel() == E, "the correction holds one number per expert");
     Tensor w = at::empty({N, top}, logits.options()), idx = at::empty({N, top}, logits.options().dtype(at::kLong));
     Tensor ident = at::empty({N}, logits.options());
-    bool ok = seqmix::route_topk(logits.data_ptr<float>(), correction ? f32(*correction) : nullptr, N, E, (int)top, (int)n_real, (int)kind,
-                                 (float)scale, w.data_ptr<float>(), idx.data_ptr<int64_t>(), ident.data_ptr<float>(), stream());
-    TORCH_CHECK(ok, "route_topk: at most 256 experts and top <= experts");
+    bool ok = seqmix::route_topk(logits.data_ptr<float>(), logits.size(1), correction ? f32(*correction) : nullptr, N, E, (int)top, (int)n_real, (int)kind,
+                                 (float)scale, (int)groups, (int)gkeep, norm, share, w.data_ptr<float>(), idx.data_ptr<int64_t>(), ident.data_ptr<float>(), stream());
+    TORCH_CHECK(ok, "route_topk: at most 256 experts, top <= experts, equal groups that leave enough to choose from");
     check_launch();
     return {w, idx, ident};
 }
@@ -248,6 +289,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("silu_mul", &silu_mul);
     m.def("indexed_gemv", &indexed_gemv);
     m.def("moe_combine", &moe_combine);
+    m.def("residual_norm_", &residual_norm_);
+    m.def("sigmoid_gate_heads", &sigmoid_gate_heads);
     m.def("embed_sinusoid", &embed_sinusoid);
     m.def("group_rms_norm_gated", &group_rms_norm_gated);
 }

@@ -2,8 +2,9 @@
 // One block = kChunk consecutive ring rows of one sequence x one tile of kHeads heads.  The block stages its ring rows in shared
 // memory once (as floats) and uses them twice: as keys (scores of every head of the tile against every row; all heads share the
 // rows) and as values (the weighted sum of the latents).  Each block leaves a partial softmax (running maximum, sum of weights,
-// unnormalised weighted sum) per head; a second kernel merges the partials of a sequence's chunks and writes the result in the
-// activation dtype.  Scores, weights and sums are float throughout.
+// unnormalised weighted sum) per head; a second kernel merges the partials of a sequence's chunks, adds the sink's exp(sink_h) to the
+// denominator (if any) and writes the result in the activation dtype.  Scores, weights and sums are float throughout.  bfloat16 rows of
+// fitting sizes take the tensor-core form of the first kernel (latent_decode_mma.cu); the merge is the same.
 // Ring row kk of a sequence at position p holds position j = p - ((p - kk) mod ring); it is visible when j >= 0 and p - j < window.
 #include "seq_common.cuh"
 #include "seqmix.h"
@@ -41,8 +42,7 @@ latent_ring_partial_kernel(const T* __restrict__ qa, long qa_sn, long qa_sh, con
     const unsigned vismask = __ballot_sync(0xffffffffu, lens[b] > 0 && lane < nr && visible(r0 + lane));
     const bool any = vismask != 0u;
     if (!any) {                                // nothing to see here: an empty partial with weight zero
-        if (tid < nh) { part_m[pbase + tid] = -INFINITY; part_l[pbase + tid] = 0.f; }
-        for (int i = tid; i < nh * C; i += kThreads) part_acc[pbase * C + i] = 0.f;
+        if (tid < nh) { part_m[pbase + tid] = -INFINITY; part_l[pbase + tid] = 0.f; }      // its sums are never read
         return;
     }
     const T* base = keys + (long)(key_index ? key_index[b] : b) * key_sb + (long)r0 * CR;
@@ -147,6 +147,7 @@ latent_ring_partial_kernel(const T* __restrict__ qa, long qa_sn, long qa_sh, con
 #pragma unroll
         for (int h = 0; h < kHeads; ++h) acc[e][h] = 0.f;
     for (int j = 0; j < nr; ++j) {
+        if (!((vismask >> j) & 1u)) continue;     // weight zero: whatever the row holds
         float kv[kColsPerThread];
 #pragma unroll
         for (int e = 0; e < kColsPerThread; ++e) {
@@ -178,14 +179,14 @@ latent_ring_partial_kernel(const T* __restrict__ qa, long qa_sn, long qa_sh, con
 // formed once (a lane per chunk) and kept in shared memory; every thread then sums its columns over the chunks, loads unrolled.
 template <typename T>
 __global__ void latent_ring_merge_kernel(const float* __restrict__ part_m, const float* __restrict__ part_l,
-                                         const float* __restrict__ part_acc, int nsplit, int H, int C, T* __restrict__ out, long out_sn,
-                                         long out_sh) {
+                                         const float* __restrict__ part_acc, int nsplit, int H, int C, const float* __restrict__ sink,
+                                         T* __restrict__ out, long out_sn, long out_sh) {
     extern __shared__ float sw[];              // [nsplit]
     __shared__ float red[2];
     const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
     const long i0 = (long)b * nsplit * H + h;  // partial of chunk s: i0 + s * H
     if (tid < 32) {
-        float M = -INFINITY;
+        float M = sink ? sink[h] : -INFINITY;
         for (int s = lane; s < nsplit; s += 32) M = fmaxf(M, part_m[i0 + (long)s * H]);
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
@@ -197,6 +198,7 @@ __global__ void latent_ring_merge_kernel(const float* __restrict__ part_m, const
             L = fmaf(l, w, L);
         }
         L = warp_sum(L);
+        if (sink) L += expf(sink[h] - M);
         if (lane == 0) { red[0] = M; red[1] = L; }
     }
     __syncthreads();
@@ -210,7 +212,8 @@ __global__ void latent_ring_merge_kernel(const float* __restrict__ part_m, const
         const float* pa = part_acc + i0 * C + c;
         float a = 0.f;
 #pragma unroll 8
-        for (int s = 0; s < nsplit; ++s) a = fmaf(pa[(long)s * H * C], sw[s], a);
+        for (int s = 0; s < nsplit; ++s)
+            if (sw[s] > 0.f) a = fmaf(pa[(long)s * H * C], sw[s], a);      // chunks that saw nothing left no sums
         stf(o + c, a * inv);
     }
 }
@@ -224,8 +227,7 @@ bool latent_ring_decode_fits(int C, int R) {
 template <typename T>
 static void ring_decode_launch(const void* qa, long qa_sn, long qa_sh, const void* qr, long qr_sn, long qr_sh, const void* keys, long key_sb,
                                int ring, const int* key_index, const int* pos0, const int* lens, int B, int H, int C, int R, int window,
-                               float scale, float* part_m, float* part_l, float* part_acc, void* out, long out_sn, long out_sh,
-                               cudaStream_t s) {
+                               float scale, float* part_m, float* part_l, float* part_acc, cudaStream_t s) {
     const int nsplit = latent_ring_decode_splits(ring);
     const size_t smem = (size_t)((kHeads + kChunk) * ((C + R + 31) & ~31) + 2 * kHeads * kChunk) * sizeof(float);
     dim3 grid(nsplit, B, (H + kHeads - 1) / kHeads);
@@ -241,18 +243,30 @@ static void ring_decode_launch(const void* qa, long qa_sn, long qa_sh, const voi
     } while (0)
     if (vec) SEQMIX_RING(true); else SEQMIX_RING(false);
 #undef SEQMIX_RING
+}
+
+template <typename T>
+static void ring_merge_launch(const float* part_m, const float* part_l, const float* part_acc, int nsplit, int B, int H, int C, const float* sink,
+                              void* out, long out_sn, long out_sh, cudaStream_t s) {
     const int mt = C >= 256 ? 256 : (C >= 128 ? 128 : 64);
-    latent_ring_merge_kernel<T><<<dim3(H, B), mt, nsplit * sizeof(float), s>>>(part_m, part_l, part_acc, nsplit, H, C, (T*)out, out_sn, out_sh);
+    const size_t smem = nsplit * sizeof(float);
+    if (smem > 48 * 1024) cudaFuncSetAttribute(latent_ring_merge_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    latent_ring_merge_kernel<T><<<dim3(H, B), mt, smem, s>>>(part_m, part_l, part_acc, nsplit, H, C, sink, (T*)out, out_sn, out_sh);
 }
 
 void latent_ring_decode(const void* qa, int bf, long qa_sn, long qa_sh, const void* qr, long qr_sn, long qr_sh, const void* keys,
                         long key_sb, int ring, const int* key_index, const int* pos0, const int* lens, int B, int H, int C, int R,
-                        int window, float scale, float* part_m, float* part_l, float* part_acc, void* out, long out_sn, long out_sh,
-                        cudaStream_t s) {
-    if (bf) ring_decode_launch<bf16>(qa, qa_sn, qa_sh, qr, qr_sn, qr_sh, keys, key_sb, ring, key_index, pos0, lens, B, H, C, R, window, scale,
-                                     part_m, part_l, part_acc, out, out_sn, out_sh, s);
+                        int window, float scale, const float* sink, int mma, int nsplit, float* part_m, float* part_l, float* part_acc,
+                        void* out, long out_sn, long out_sh, cudaStream_t s) {
+    if (mma)
+        latent_decode_mma(qa, qa_sn, qa_sh, qr, qr_sn, qr_sh, keys, key_sb, ring, key_index, pos0, lens, B, H, C, R, window, scale, nsplit,
+                          part_m, part_l, part_acc, s);
+    else if (bf) ring_decode_launch<bf16>(qa, qa_sn, qa_sh, qr, qr_sn, qr_sh, keys, key_sb, ring, key_index, pos0, lens, B, H, C, R, window, scale,
+                                     part_m, part_l, part_acc, s);
     else ring_decode_launch<float>(qa, qa_sn, qa_sh, qr, qr_sn, qr_sh, keys, key_sb, ring, key_index, pos0, lens, B, H, C, R, window, scale,
-                                   part_m, part_l, part_acc, out, out_sn, out_sh, s);
+                                   part_m, part_l, part_acc, s);
+    if (bf) ring_merge_launch<bf16>(part_m, part_l, part_acc, nsplit, B, H, C, sink, out, out_sn, out_sh, s);
+    else ring_merge_launch<float>(part_m, part_l, part_acc, nsplit, B, H, C, sink, out, out_sn, out_sh, s);
 }
 
 }  // namespace seqmix

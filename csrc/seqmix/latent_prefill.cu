@@ -5,7 +5,8 @@
 // share (from the prepared latent rows).  Scores come from
 // tensor-core products (mma.sync m16n8k16, float accumulation), are scaled, masked and exponentiated in float with a running maximum
 // and sum per query; the weights are rounded to bfloat16 only as operands of the value product, whose accumulator is float.
-// Position i sees j with 0 <= i - j < window.  Queries at or past lens[b] give zeros.
+// Position i sees j with 0 <= i - j < window.  Queries at or past lens[b] give zeros.  With `sink` the softmax denominator also holds
+// exp(sink_h); with `gate` the results are multiplied by sigmoid(gate) per coordinate on their way out.
 // Sizes: key and value sizes are multiples of 16 up to 16 * DK16 / 16 * VD16 (template bounds; the real sizes are arguments).
 #include "mma_tiles.cuh"
 #include "seq_common.cuh"
@@ -19,9 +20,9 @@ constexpr int kQT = 64, kKT = 64, kPad = 8;     // queries / keys per tile; row 
 // out [B,S,H*VD].  DK = D + R.
 template <int DK16, int VD16>
 __global__ void __launch_bounds__(128)
-latent_prompt_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kx, const bf16* __restrict__ rows, const bf16* __restrict__ v,
+latent_prompt_attn_kernel(const bf16* __restrict__ q, long q_sn, const bf16* __restrict__ kx, const bf16* __restrict__ rows, const bf16* __restrict__ v,
                           const int* __restrict__ lens, int S, int H, int D, int R, int CR, int VD, int window, float scale,
-                          bf16* __restrict__ out) {
+                          const float* __restrict__ sink, const bf16* __restrict__ gate, long gate_sn, bf16* __restrict__ out) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int DK = D + R, dk16 = DK / 16, vd16 = VD / 16, ldk = DK + kPad, ldv = VD + kPad;
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);          // [kQT][ldk] queries, then key stage 1 (same size)
@@ -41,7 +42,7 @@ latent_prompt_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
     // queries of the tile (rows past the sequence: zeros)
     for (int i = tid; i < kQT * (DK / 8); i += 128) {
         const int r = i / (DK / 8), c = (i % (DK / 8)) * 8, t = q0 + r;
-        *reinterpret_cast<uint4*>(Qs + r * ldk + c) = t < S ? *reinterpret_cast<const uint4*>(q + (((long)b * S + t) * H + h) * DK + c) : zero4;
+        *reinterpret_cast<uint4*>(Qs + r * ldk + c) = t < S ? *reinterpret_cast<const uint4*>(q + ((long)b * S + t) * q_sn + (long)h * DK + c) : zero4;
     }
     __syncthreads();
     const int r0 = warp * 16, g = lane >> 2, tq = lane & 3;
@@ -169,13 +170,32 @@ latent_prompt_attn_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
         lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 1);
         lrow[r] += __shfl_xor_sync(0xffffffffu, lrow[r], 2);
     }
-    const float inv0 = (i0 < len && lrow[0] > 0.f) ? 1.f / lrow[0] : 0.f, inv1 = (i1 < len && lrow[1] > 0.f) ? 1.f / lrow[1] : 0.f;
+    float grow[2] = {1.f, 1.f};                            // what a sink above the keys' maximum does to sums relative to that maximum
+    if (sink) {
+        const float sk = sink[h] * 1.4426950408889634f;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const float m = fmaxf(mrow[r], sk);
+            grow[r] = exp2f(mrow[r] - m);
+            lrow[r] = lrow[r] * grow[r] + exp2f(sk - m);
+        }
+    }
+    const float inv0 = (i0 < len && lrow[0] > 0.f) ? grow[0] / lrow[0] : 0.f, inv1 = (i1 < len && lrow[1] > 0.f) ? grow[1] / lrow[1] : 0.f;
+    const bf16* gb = gate ? gate + (long)b * S * gate_sn + (long)h * VD : nullptr;
+    auto gated = [&](int i, int c, float a, float d) -> unsigned {
+        if (gb && i < len) {
+            const __nv_bfloat162 z = *reinterpret_cast<const __nv_bfloat162*>(gb + (long)i * gate_sn + c);
+            a *= sigmoidf_(__low2float(z));
+            d *= sigmoidf_(__high2float(z));
+        }
+        return pack2(a, d);
+    };
 #pragma unroll
     for (int n = 0; n < 2 * VD16; ++n) {
         if (n < 2 * vd16) {
             const int c = n * 8 + tq * 2;
-            if (i0 < S) *reinterpret_cast<unsigned*>(ob + (long)i0 * H * VD + c) = pack2(oacc[n][0] * inv0, oacc[n][1] * inv0);
-            if (i1 < S) *reinterpret_cast<unsigned*>(ob + (long)i1 * H * VD + c) = pack2(oacc[n][2] * inv1, oacc[n][3] * inv1);
+            if (i0 < S) *reinterpret_cast<unsigned*>(ob + (long)i0 * H * VD + c) = gated(i0, c, oacc[n][0] * inv0, oacc[n][1] * inv0);
+            if (i1 < S) *reinterpret_cast<unsigned*>(ob + (long)i1 * H * VD + c) = gated(i1, c, oacc[n][2] * inv1, oacc[n][3] * inv1);
         }
     }
 }
@@ -185,8 +205,9 @@ bool latent_prompt_attention_fits(int D, int R, int CR, int VD) {
     return DK % 16 == 0 && VD % 16 == 0 && D % 8 == 0 && R % 8 == 0 && CR % 8 == 0 && DK <= 256 && VD <= 256;
 }
 
-bool latent_prompt_attention(const void* q, const void* kx, const void* rows, const void* v, const int* lens, int B, int S, int H, int D,
-                             int R, int CR, int VD, int window, float scale, void* out, cudaStream_t s) {
+bool latent_prompt_attention(const void* q, long q_sn, const void* kx, const void* rows, const void* v, const int* lens, int B, int S, int H,
+                             int D, int R, int CR, int VD, int window, float scale, const float* sink, const void* gate, long gate_sn,
+                             void* out, cudaStream_t s) {
     if (!latent_prompt_attention_fits(D, R, CR, VD)) return false;
     const int DK = D + R;
     const size_t smem = (size_t)((kQT + kKT) * (DK + kPad) + 2 * kKT * (VD + kPad)) * sizeof(bf16);
@@ -194,8 +215,8 @@ bool latent_prompt_attention(const void* q, const void* kx, const void* rows, co
 #define SEQMIX_LPA(A, Bv)                                                                                                           \
     do {                                                                                                                            \
         cudaFuncSetAttribute(latent_prompt_attn_kernel<A, Bv>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);            \
-        latent_prompt_attn_kernel<A, Bv><<<grid, 128, smem, s>>>((const bf16*)q, (const bf16*)kx, (const bf16*)rows, (const bf16*)v, lens, \
-                                                                S, H, D, R, CR, VD, window, scale, (bf16*)out);                     \
+        latent_prompt_attn_kernel<A, Bv><<<grid, 128, smem, s>>>((const bf16*)q, q_sn, (const bf16*)kx, (const bf16*)rows, (const bf16*)v, lens, \
+                                                                S, H, D, R, CR, VD, window, scale, sink, (const bf16*)gate, gate_sn, (bf16*)out);                     \
     } while (0)
     if (DK <= 64 && VD <= 64) SEQMIX_LPA(4, 4);
     else if (DK <= 128 && VD <= 128) SEQMIX_LPA(8, 8);

@@ -7,32 +7,48 @@ namespace seqmix {
 void short_conv(const void* x, int in_bf16, long x_sb, long x_st, const float* w, const float* bias, void* state, const int* slots,
                 const int* lens, int B, int S, int C, int taps, int fresh, int residual, int act, void* out, int out_bf16, cudaStream_t s);
 void rms_norm(const void* x, int in_bf16, long x_stride, int rows, int C, const float* w, int w_stride, float eps, const void* gate,
-              long gate_stride, void* out, int out_bf16, long out_stride, float* res, long res_stride, int center, cudaStream_t s);
+              long gate_stride, void* out, int out_bf16, long out_stride, float* res, long res_stride, int center, const float* bias,
+              cudaStream_t s);
+// x (float, in place) += scale * y, then (w given) h <- norm(x) * w + bias; y [rows, C], or with top > 0 the expert rows whose weighted
+// sums (weight, src [rows, top]; base times base_weight added) take its place.  scale, bias, base, base_weight, w may be null.
+void residual_norm(float* x, long x_stride, const void* y, long y_stride, int bf, const int* src, const float* weight, int top, const void* base,
+                   const float* base_weight, const float* scale, const float* w, const float* bias, float eps, int center, int rows, int C,
+                   void* h, long h_stride, cudaStream_t s);
 // x (float, in place) <- norm(alpha * x + sigmoid(gate) * y) * w; gate may be null; lp (of y's dtype, may be null) gets a copy
 void postnorm_gated(float* x, long x_stride, const void* y, long y_stride, const void* gate, long gate_stride, int bf, const float* w,
                     float alpha, float eps, int rows, int C, void* lp, long lp_stride, cudaStream_t s);
 void latent_kv_store(const void* kv, int bf, long kv_sb, long kv_st, int B, int S, int C, int R, int dims, const float* nw, float eps,
                      const float* inv_freq, const int* pos0, const int* lens, const int* slots, void* cache, int ring, void* rows,
-                     cudaStream_t s);
-void rope_q(void* q, int bf, long q_sn, long q_sh, int N, int S, int H, int dims, const float* inv_freq, const int* pos0, cudaStream_t s);
+                     float amp, void* q, long q_sn, long q_sh, int H, cudaStream_t s);       // q (optional): H heads rotated in place
+void rope_q(void* q, int bf, long q_sn, long q_sh, int N, int S, int H, int dims, const float* inv_freq, const int* pos0, float amp,
+            cudaStream_t s);
 void latent_window_attention(const void* qa, int bf, long qa_sn, long qa_sh, const void* qr, long qr_sn, long qr_sh, const void* keys,
                              long key_sb, int ring, const int* key_index, const int* pos0, const int* lens, int B, int S, int H, int C,
-                             int R, int window, float scale, void* out, long out_sn, long out_sh, cudaStream_t s);
+                             int R, int window, float scale, const float* sink, void* out, long out_sn, long out_sh, cudaStream_t s);
 // Single new tokens against their rings (latent_decode.cu): blocks over (ring chunk, sequence, head tile) leave partial softmaxes
 // part_m / part_l [B, splits, H] and part_acc [B, splits, H, C] (float), which a second kernel merges into out[h, b, :].
 int latent_ring_decode_splits(int ring);
 bool latent_ring_decode_fits(int C, int R);
 void latent_ring_decode(const void* qa, int bf, long qa_sn, long qa_sh, const void* qr, long qr_sn, long qr_sh, const void* keys,
                         long key_sb, int ring, const int* key_index, const int* pos0, const int* lens, int B, int H, int C, int R,
-                        int window, float scale, float* part_m, float* part_l, float* part_acc, void* out, long out_sn, long out_sh,
-                        cudaStream_t s);
+                        int window, float scale, const float* sink, int mma, int nsplit, float* part_m, float* part_l, float* part_acc,
+                        void* out, long out_sn, long out_sh, cudaStream_t s);
+// The tensor-core form of the first kernel (latent_decode_mma.cu; bfloat16, C and R in whole 16s): a sequence's visible rows are cut
+// into `nsplit` stretches whatever the ring's length.  `latent_ring_decode` with `mma` set runs it and the merge.
+bool latent_decode_mma_fits(int C, int R);
+int latent_decode_mma_splits(int B, int H, int rows);
+void latent_decode_mma(const void* qa, long qa_sn, long qa_sh, const void* qr, long qr_sn, long qr_sh, const void* keys, long key_sb, int ring,
+                       const int* key_index, const int* pos0, const int* lens, int B, int H, int C, int R, int window, float scale,
+                       int nsplit, float* part_m, float* part_l, float* part_acc, cudaStream_t s);
 // Prompt attention in the expanded form as one fused kernel (latent_prefill.cu; bfloat16, sizes in whole 16s up to 256): q [B,S,H,D+R],
-// kx [B,S,H,D], rows [B,S,CR] (last R numbers: the shared rotated key part), v [B,S,H,VD] → out [B,S,H*VD].  false: sizes do not fit.
+// kx [B,S,H,D], rows [B,S,CR] (last R numbers: the shared rotated key part), v [B,S,H,VD] → out [B,S,H*VD].  q_sn: elements between
+// tokens of q; sink (one per head) and gate (pre-sigmoid, [B*S, >= H*VD], row stride gate_sn) may be null.  false: sizes do not fit.
 bool latent_prompt_attention_fits(int D, int R, int CR, int VD);
-bool latent_prompt_attention(const void* q, const void* kx, const void* rows, const void* v, const int* lens, int B, int S, int H, int D,
-                             int R, int CR, int VD, int window, float scale, void* out, cudaStream_t s);
+bool latent_prompt_attention(const void* q, long q_sn, const void* kx, const void* rows, const void* v, const int* lens, int B, int S, int H,
+                             int D, int R, int CR, int VD, int window, float scale, const float* sink, const void* gate, long gate_sn,
+                             void* out, cudaStream_t s);
 void window_softmax(const float* scores, long rows, int span, float scale, int ring_mode, int H, int Qb, int nblk, int w_eff, int window,
-                    const int* pos0, const int* lens, void* out, int out_bf16, cudaStream_t s);
+                    const int* pos0, const int* lens, const float* sink, int nsink, void* out, int out_bf16, cudaStream_t s);
 // `decay` (one float per head, or null): a fixed decay per head instead of the projected z (retention); z and zbias are not read then.
 bool gla_scan(const void* q, const void* k, const void* v, int bf, long sb, long st, const void* z, long z_sb, long z_st,
               const float* zbias, float inv_tau, float qscale, const float* decay, float* state, const int* slots, const int* lens,
@@ -70,8 +86,9 @@ void indexed_gemv(const void* w, const int* sel, const void* x, int bf, long x_s
 void moe_combine(const void* rows, const int* src, const float* weight, const void* base, const float* base_weight, int bf, int N, int top,
                  int C, void* out, cudaStream_t s);
 // false: more experts than the kernel takes (256)
-bool route_topk(const float* logits, const float* correction, int N, int E, int top, int n_real, int kind, float scale, float* w, long* idx,
-                float* ident, cudaStream_t s);
+bool route_topk(const float* logits, long z_stride, const float* correction, int N, int E, int top, int n_real, int kind, float scale, int groups,
+                int gkeep, int norm, int share, float* w, long* idx, float* ident, cudaStream_t s);
+void sigmoid_gate_heads(const void* ov, const void* gate, long gate_stride, int bf, long N, int H, int V, void* out, cudaStream_t s);
 void small_linear_f32(const void* w, int w_bf, const void* x, int x_bf, long x_stride, int N, int O, int I, float* out, cudaStream_t s);
 void embed_sinusoid(const long* tokens, const void* table, int bf, float scale, const float* inv_freq, const int* pos0, int B, int S, int W,
                     int vocab, float* out, cudaStream_t s);

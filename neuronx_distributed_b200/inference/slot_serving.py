@@ -2,6 +2,9 @@
 function over any rows and slots (``forward_step`` → float residual stream, ``logits``), and on top of it the static-batch entry
 points of ``LlamaForInference`` (``context_encoding`` / ``token_generation`` / ``generate``) with the framework's sampler.
 
+A language model whose layers keep whole sequences (no window) names the longest one its caches hold as ``position_limit``; a step that
+would pass it is refused wherever the positions are known on the host.
+
 A family provides a language model with ``embed`` (a parameter, for the device), ``state_specs()``,
 ``body(input_ids, ctx, states, tap)`` → float ``[B,S,width]`` and ``logits(rows)``; the subclass adds ``from_pretrained`` and
 ``load_checkpoint_tensors``."""
@@ -51,8 +54,18 @@ class SlotServingModel(nn.Module):
         layer.  ``fresh``: the rows start new sequences (prompts); otherwise they continue from their slots' state."""
         if not fresh and input_ids.shape[1] != 1:
             raise ValueError("a continuing step carries one token per row")
+        self._check_room(lens, pos0, input_ids.shape[1] if fresh else 1)
         ctx = StepContext(self._i32(lens), self._i32(slots), self._i32(pos0), bool(fresh))
         return self.lm.body(input_ids, ctx, self.states, tap)
+
+    def _check_room(self, lens, pos0, longest: int) -> None:
+        limit = getattr(self.lm, "position_limit", None)
+        if limit is None:
+            return
+        on_host = not isinstance(lens, torch.Tensor) and not isinstance(pos0, torch.Tensor)
+        end = max((int(n) + int(p) for n, p in zip(lens, pos0)), default=0) if on_host else longest
+        if end > limit:
+            raise ValueError(f"position {end - 1} is beyond the cache of {limit} tokens per sequence")
 
     def logits(self, rows: torch.Tensor) -> torch.Tensor:
         return self.lm.logits(rows)
@@ -93,6 +106,7 @@ class SlotServingModel(nn.Module):
     def generate(self, prompt_ids: torch.Tensor, max_new_tokens: int, prompt_lens: Optional[torch.Tensor] = None) -> torch.Tensor:
         B, S = prompt_ids.shape
         lens = prompt_lens if prompt_lens is not None else torch.full((B,), S, device=prompt_ids.device, dtype=torch.long)
+        self._check_room([int(lens.max())], [max(0, max_new_tokens - 1)], S)
         tok = self.context_encoding(prompt_ids, lens - 1)
         out, pos = [tok], lens.clone()
         for _ in range(max_new_tokens - 1):

@@ -8,6 +8,11 @@ over the up rows in ``up [E, 2 ff, width]``; ``down [E, width, ff]``.
 (renormalised by construction).  ``router_bias``: the logits are ``W_router h + b``.  ``expert_act``: the plain experts' activation,
 ``"gelu"`` (erf form) or ``"relu_sq"`` (the square of relu).
 
+``groups = (count, keep)``: the choice is limited to the ``keep`` best of ``count`` equal groups of neighbouring experts (a group is
+worth the sum of its two largest scores).  ``renormalise``: the chosen scores are divided by their sum.  ``shared_gated``: the shared
+expert has the gated form (``shared_up [2 shared_ff, width]``: gate rows over up rows).  ``shared_gate``: the shared expert's output is
+multiplied by ``sigmoid(w . h)``, one number per token; that row rides on the router's product as its last one.
+
 Two more options of the router.  ``choice_bias``: a float vector added to the scores for the CHOICE only (the weights stay the plain
 scores).  ``identity_experts``: the router's last outputs name experts without tensors whose output is the input itself; their
 weights are summed per token and enter the combine as a weighted copy of the input.
@@ -35,14 +40,17 @@ class RoutedFFN(nn.Module):
 
     def __init__(self, width: int, ff: int, experts: int, top: int, weight_scale: float = 1.0, shared_ff: int = 0,
                  router_act: str = "sigmoid", gated: bool = False, identity_experts: int = 0, choice_bias: bool = False,
-                 dtype: torch.dtype = torch.bfloat16, device=None, router_bias: bool = False, expert_act: str = "gelu"):
+                 dtype: torch.dtype = torch.bfloat16, device=None, router_bias: bool = False, expert_act: str = "gelu",
+                 groups=None, renormalise: bool = False, shared_gated: bool = False, shared_gate: bool = False):
         super().__init__()
+        assert not shared_gate or (shared_ff and not identity_experts), "a gate needs a shared expert (and identity experts take its place)"
         assert expert_act in ("gelu", "relu_sq"), expert_act
         assert router_act != "softmax_top" or not (identity_experts or choice_bias), "softmax over the chosen logits: plain experts only"
         self.expert_act = expert_act
         self.width, self.ff, self.experts, self.top, self.weight_scale, self.shared_ff = width, ff, experts, top, weight_scale, shared_ff
         self.gated, self.identity_experts = gated, identity_experts
-        self.router = RouterTopK(experts + identity_experts, top, width, dtype=torch.float32, device=device, bias=router_bias,
+        self.groups, self.renormalise, self.shared_gated, self.shared_gate = groups, renormalise, shared_gated, shared_gate
+        self.router = RouterTopK(experts + identity_experts + int(shared_gate), top, width, dtype=torch.float32, device=device, bias=router_bias,
                                  act_fn="softmax" if router_act == "softmax_top" else router_act,
                                  apply_act_fn_over_topk=router_act == "softmax_top")
         self.router_act = router_act
@@ -52,7 +60,7 @@ class RoutedFFN(nn.Module):
         self.correction = nn.Parameter(torch.zeros(experts + identity_experts, dtype=torch.float32, device=device),
                                        requires_grad=False) if choice_bias else None
         if shared_ff:
-            self.shared_up, self.shared_down = mk(shared_ff, width), mk(width, shared_ff)
+            self.shared_up, self.shared_down = mk((2 if shared_gated else 1) * shared_ff, width), mk(width, shared_ff)
         self._router_lowp = None       # (version of the router matrix, its bfloat16 transpose or None when that would round)
 
     def _router_logits(self, h: torch.Tensor) -> torch.Tensor:
@@ -77,11 +85,11 @@ class RoutedFFN(nn.Module):
         return seqmix.matmul_f32(h[None], self._router_lowp[1][None])[0]
 
     def route(self, h: torch.Tensor):
-        """Float scores of all experts → (weights ``[N, top]`` float, expert ids ``[N, top]``, identity share ``[N]`` float or None):
-        one kernel for scores, correction, top-k and the identity experts' share (``seqmix.route_topk``)."""
+        """Float scores of all experts → (weights ``[N, top]`` float, expert ids ``[N, top]``, identity share or shared expert's gate
+        ``[N]`` float, or None): one kernel for scores, correction, groups, top-k and that number (``seqmix.route_topk``)."""
         w, idx, ident = seqmix.route_topk(self._router_logits(h), self.correction, self.top, self.experts, self.router_act,
-                                          self.weight_scale)
-        return w, idx, (ident if self.identity_experts else None)
+                                          self.weight_scale, self.groups, self.renormalise, self.shared_gate)
+        return w, idx, (ident if self.identity_experts or self.shared_gate else None)
 
     def _act(self, y: torch.Tensor) -> torch.Tensor:
         """The experts' activation on the up-projection's output: ``[M, ff]`` (plain) or ``[M, 2 ff]`` → ``[M, ff]`` (gated)."""
@@ -130,6 +138,12 @@ class RoutedFFN(nn.Module):
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         """``h [N, width]`` → ``[N, width]``."""
+        rows, (src, w, base, base_w) = self.pieces(h)
+        return seqmix.moe_combine(rows, src, w, base, base_w)
+
+    def pieces(self, h: torch.Tensor):
+        """``h [N, width]`` → ``(expert rows [M, width], (src, weights, base, base weights))``: what ``moe_combine`` (or a residual sum that
+        does its work, ``seqmix.residual_norm_``) adds up."""
         N = h.shape[0]
         w, idx, ident_w = self.route(h)                            # identity choices: weight 0, their scores summed in ident_w
         M = N * self.top
@@ -158,6 +172,9 @@ class RoutedFFN(nn.Module):
         if self.identity_experts:
             if self.shared_ff:
                 raise NotImplementedError("identity experts together with a shared expert")
-            return seqmix.moe_combine(eo, src, w.contiguous(), h, ident_w)
-        base = F.linear(seqmix.gelu_erf(F.linear(h, self.shared_up)), self.shared_down) if self.shared_ff else None
-        return seqmix.moe_combine(eo, src, w.contiguous(), base)
+            return eo, (src, w.contiguous(), h, ident_w)
+        base = None
+        if self.shared_ff:
+            mid = F.linear(h, self.shared_up)
+            base = F.linear(seqmix.silu_mul(mid) if self.shared_gated else seqmix.gelu_erf(mid), self.shared_down)
+        return eo, (src, w.contiguous(), base, ident_w if self.shared_gate else None)

@@ -134,6 +134,30 @@ class GainOnlyLayerNorm(nn.Module):
         return res
 
 
+class AffineLayerNorm(nn.Module):
+    """Layer norm with a gain and a bias, statistics in float, float parameters: ``(x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b``.
+    ``forward`` gives a sublayer's input in ``out_dtype``; ``after_sum`` is the same norm joined with the residual sum before it: the
+    float stream gets ``x += scale * y`` in place (``scale``: one float per coordinate) and the new rows' norm comes back in ``y``'s
+    dtype, one kernel (``csrc/seqmix/norms.cu``).  ``experts``: see ``ops.seqmix.residual_norm_``."""
+
+    def __init__(self, width: int, eps: float = 1e-6, device=None):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(width, dtype=torch.float32, device=device), requires_grad=False)
+        self.bias = nn.Parameter(torch.zeros(width, dtype=torch.float32, device=device), requires_grad=False)
+        self.eps = eps
+
+    def forward(self, input: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        from ..ops import seqmix
+
+        x = input
+        return seqmix.rms_norm(x.reshape(-1, x.shape[-1]), self.weight, self.eps, None, out_dtype or x.dtype, center=True, bias=self.bias).view(x.shape)
+
+    def after_sum(self, x: torch.Tensor, y: torch.Tensor, scale: torch.Tensor, experts=None) -> torch.Tensor:
+        from ..ops import seqmix
+
+        return seqmix.residual_norm_(x, y, scale, self.weight, self.bias, self.eps, True, experts)
+
+
 class GatedPostRMSNorm(nn.Module):
     """The closing step of a block whose norm comes AFTER the residual sum: ``x <- rms_norm(alpha * x + sigmoid(g) * y) * w`` on a
     float stream ``x`` in place, with ``y`` the sublayer's result and ``g`` the logits of a gate per coordinate (``None``: no gate) that

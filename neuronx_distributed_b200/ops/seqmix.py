@@ -1,6 +1,7 @@
-"""Sequence-mixer ops: short causal convolutions with carried history, scalar / vector RMS norms (optionally accumulated into a
-float residual stream, or closing a block whose norm follows a gated residual sum), token embeddings with sinusoids or a hashed
-pair table, latent / grouped-query / head-mixing sliding-window attention over ring caches (softmax or independent sigmoid weights),
+"""Sequence-mixer ops: short causal convolutions with carried history, scalar / vector RMS and layer norms (optionally accumulated
+into a float residual stream, closing a block whose norm follows a gated residual sum, or joined with the residual sum before them), token embeddings with sinusoids or a hashed
+pair table, latent / grouped-query / head-mixing attention over ring caches (sliding window or the whole sequence; softmax, with or
+without a sink, or independent sigmoid weights),
 gated linear recurrences (per-key-channel decay; real-gated LRU; minGRU), matrix-state recurrences, xIELU / erf-GELU / squared relu
 and the small-batch pieces of a routed feed-forward.
 
@@ -33,8 +34,8 @@ GROUPS = {
     "core": (["short_conv.cu", "norms.cu", "activations.cu", "embed.cu", "rotary.cu", "bind_core.cpp"],
              ["short_conv", "rms_norm", "add_rms_norm_", "xielu", "gelu_erf", "silu_mul", "indexed_gemv", "moe_combine", "embed_sinusoid",
               "group_rms_norm_gated", "route_topk", "small_linear_f32", "clamped_glu", "sigmoid_gate_mul_", "rotary_qkv_f32", "relu_sq",
-              "embed_bigram", "postnorm_gated_"]),
-    "latent": (["latent_attention.cu", "latent_decode.cu", "latent_prefill.cu", "bind_latent.cpp"],
+              "embed_bigram", "postnorm_gated_", "residual_norm_", "sigmoid_gate_heads"]),
+    "latent": (["latent_attention.cu", "latent_decode.cu", "latent_decode_mma.cu", "latent_prefill.cu", "bind_latent.cpp"],
                ["latent_kv_store", "rope_q_", "latent_window_attention", "window_softmax", "latent_prompt_attention",
                 "latent_prompt_attention_fits"]),
     "linrec": (["linear_recurrence.cu", "gla_chunked.cu", "bind_linrec.cpp"], ["gla_scan", "rglru_scan", "retention_scan", "mingru_scan"]),
@@ -147,18 +148,20 @@ def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], s
 
 # --------------------------------------------------------------------------------------------------------------------------- norms
 def rms_norm(x: torch.Tensor, w: torch.Tensor, eps: float, gate: Optional[torch.Tensor] = None,
-             out_dtype: Optional[torch.dtype] = None, center: bool = False) -> torch.Tensor:
+             out_dtype: Optional[torch.dtype] = None, center: bool = False, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Rows of ``x [rows, C]`` divided by their root mean square, times ``w`` (``[C]`` or one number), times ``silu(gate)``.
-    ``center``: the row's mean is taken off first (a layer norm with a gain and no bias: the statistics are the mean and the mean
-    squared deviation)."""
+    ``center``: the row's mean is taken off first (a layer norm: the statistics are the mean and the mean squared deviation);
+    ``bias [C]`` is added at the end."""
     out_dtype = out_dtype or x.dtype
     if _cuda(x):
         _ext.count_launch()
-        return ext().rms_norm(x, w, eps, gate, out_dtype == torch.bfloat16, center)
+        return ext().rms_norm(x, w, eps, gate, out_dtype == torch.bfloat16, center, bias)
     xf = x.float()
     if center:
         xf = xf - xf.mean(-1, keepdim=True)
     y = xf / torch.sqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w
+    if bias is not None:
+        y = y + bias
     if gate is not None:
         y = y * F.silu(gate.float())
     return y.to(out_dtype)
@@ -193,15 +196,45 @@ def postnorm_gated_(x: torch.Tensor, y: torch.Tensor, gate: Optional[torch.Tenso
     return x
 
 
+def residual_norm_(x: torch.Tensor, y: torch.Tensor, scale: Optional[torch.Tensor], w: Optional[torch.Tensor], bias: Optional[torch.Tensor],
+                   eps: float, center: bool = False, experts=None) -> Optional[torch.Tensor]:
+    """The joint between two sublayers of a pre-norm model, one launch: the float stream ``x [rows, C]`` gets ``x += scale * y`` in place
+    (``scale [C]`` float or None) and the new rows' norm ``norm(x) * w + bias`` comes back in ``y``'s dtype (``center``: a layer norm,
+    otherwise an RMS norm; ``w`` None: no norm, returns None).  ``experts = (src, weight, base, base_weight)``: ``y`` holds a routed
+    feed-forward's expert rows ``[M, C]`` and ``sum_k weight[n,k] * y[src[n,k]] (+ base_weight[n] * base[n])``, summed in float, takes
+    its place."""
+    src, weight, base, base_weight = experts if experts is not None else (None, None, None, None)
+    if _cuda(x):
+        _ext.count_launch()
+        h = ext().residual_norm_(x, y, scale, w, bias, float(eps), center, None if src is None else _i32(src), weight, base, base_weight)
+        return h if w is not None else None
+    v = y.float()
+    if src is not None:
+        v = (v[src.long()] * weight[..., None]).sum(1)
+        if base is not None:
+            v = v + (base.float() if base_weight is None else base.float() * base_weight[:, None])
+    x += v if scale is None else scale * v
+    return None if w is None else rms_norm(x, w, eps, None, y.dtype, center, bias)
+
+
 # ---------------------------------------------------------------------------------------------------------------- latent attention
 def rotary_inv_freq(dims: int, base: float, device=None, scaling: Optional[dict] = None) -> torch.Tensor:
     """``base^(-2i/dims)`` for i < dims/2, rounded once from float64.  ``scaling`` (``factor``, ``low``, ``high``, ``original``)
     rescales them for a longer context by wavelength ``l = 2 pi / f``: kept where ``l < original / high``, divided by ``factor`` where
     ``l > original / low``, and in between blended with ``s = (original / l - low) / (high - low)`` as
-    ``(1 - s) f / factor + s f``."""
+    ``(1 - s) f / factor + s f``.  ``scaling`` with ``fast`` and ``slow`` (``factor``, ``original``) blends by PAIR INDEX instead: the
+    pair whose wave turns ``t`` times over the original length has index ``dims ln(original / (2 pi t)) / (2 ln base)``; pairs up to
+    (the floor of) that of ``fast`` turns keep their frequency, pairs from (the ceiling of) that of ``slow`` turns on are divided by
+    ``factor``, linear in between.  The amplitude that goes with it is :func:`rotary_amplitude`."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
-    if scaling:
+    if scaling and "fast" in scaling:
+        factor, orig, fast, slow = (float(scaling[k]) for k in ("factor", "original", "fast", "slow"))
+        at = lambda turns: dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))
+        lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        f = f / factor * ramp + f * (1.0 - ramp)
+    elif scaling:
         factor, low, high, orig = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
         wl = 2.0 * math.pi / f
         s_ = (orig / wl - low) / (high - low) if high != low else torch.zeros_like(f)
@@ -209,23 +242,31 @@ def rotary_inv_freq(dims: int, base: float, device=None, scaling: Optional[dict]
     return f.float().to(device)
 
 
-def _rotate(x: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, dims: int) -> torch.Tensor:
-    """x ``[..., n]`` float, pos broadcastable to x's leading dims: rotate-half on the first ``dims`` coordinates."""
+def rotary_amplitude(scaling: Optional[dict] = None) -> float:
+    """What cos and sin are multiplied by: ``0.1 ln(factor) + 1`` with the index-blended rescaling (``fast`` / ``slow``), else 1."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and "fast" in scaling else 1.0
+
+
+def _rotate(x: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, dims: int, amp: float = 1.0) -> torch.Tensor:
+    """x ``[..., n]`` float, pos broadcastable to x's leading dims: rotate-half on the first ``dims`` coordinates, times ``amp``."""
     half = dims // 2
     ang = pos.float()[..., None] * inv_freq
-    c, s = torch.cos(ang), torch.sin(ang)
+    c, s = torch.cos(ang) * amp, torch.sin(ang) * amp
     u, v = x[..., :half], x[..., half:dims]
     return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], -1)
 
 
 def latent_kv_store(kv: torch.Tensor, nw: torch.Tensor, eps: float, inv_freq: torch.Tensor, dims: int, pos0: torch.Tensor,
-                    lens: torch.Tensor, slots: torch.Tensor, cache: Optional[torch.Tensor], want_rows: bool) -> Optional[torch.Tensor]:
+                    lens: torch.Tensor, slots: torch.Tensor, cache: Optional[torch.Tensor], want_rows: bool, q: Optional[torch.Tensor] = None,
+                    q_off: int = 0, amp: float = 1.0) -> Optional[torch.Tensor]:
     """``kv [B,S,C+R]``: RMS-norm (weight ``nw [C]``) of the first C numbers, rotation of the next ``dims`` at positions
     ``pos0[b] + t``.  The last ``ring`` real tokens of each row go to ``cache [slots, ring, C+R]`` at row ``position mod ring``;
-    with ``want_rows`` the prepared rows come back as ``[B,S,C+R]``."""
+    with ``want_rows`` the prepared rows come back as ``[B,S,C+R]``.  ``q [B,S,H,Dq]`` (optional): coordinates ``[q_off, q_off+dims)`` of
+    its heads are rotated in place in the same launch (real tokens only).  ``amp`` multiplies cos and sin."""
     if _cuda(kv):
         _ext.count_launch()
-        rows = ext().latent_kv_store(kv, nw, eps, inv_freq, dims, _i32(pos0), _i32(lens), _i32(slots), cache, want_rows)
+        rows = ext().latent_kv_store(kv, nw, eps, inv_freq, dims, _i32(pos0), _i32(lens), _i32(slots), cache, want_rows, q, q_off,
+                                     float(amp))
         return rows if want_rows else None
     B, S, _ = kv.shape
     C = nw.numel()
@@ -233,7 +274,9 @@ def latent_kv_store(kv: torch.Tensor, nw: torch.Tensor, eps: float, inv_freq: to
     c = f[..., :C]
     c = c / torch.sqrt(c.pow(2).mean(-1, keepdim=True) + eps) * nw
     pos = pos0.long()[:, None] + torch.arange(S)[None, :]
-    rows = torch.cat([c, _rotate(f[..., C:], pos, inv_freq, dims)], -1).to(kv.dtype)
+    rows = torch.cat([c, _rotate(f[..., C:], pos, inv_freq, dims, amp)], -1).to(kv.dtype)
+    if q is not None:
+        rope_q_(q, q_off, dims, inv_freq, pos0, amp)
     if cache is not None:
         ring = cache.shape[1]
         for b in range(B):
@@ -243,15 +286,16 @@ def latent_kv_store(kv: torch.Tensor, nw: torch.Tensor, eps: float, inv_freq: to
     return rows if want_rows else None
 
 
-def rope_q_(q: torch.Tensor, off: int, dims: int, inv_freq: torch.Tensor, pos0: torch.Tensor) -> torch.Tensor:
-    """``q [B,S,H,Dq]``: coordinates ``[off, off+dims)`` of every head rotated in place at positions ``pos0[b] + t``."""
+def rope_q_(q: torch.Tensor, off: int, dims: int, inv_freq: torch.Tensor, pos0: torch.Tensor, amp: float = 1.0) -> torch.Tensor:
+    """``q [B,S,H,Dq]``: coordinates ``[off, off+dims)`` of every head rotated in place at positions ``pos0[b] + t``
+    (cos and sin times ``amp``)."""
     if _cuda(q):
         _ext.count_launch()
-        ext().rope_q_(q, off, dims, inv_freq, _i32(pos0))
+        ext().rope_q_(q, off, dims, inv_freq, _i32(pos0), float(amp))
         return q
     S = q.shape[1]
     pos = (pos0.long()[:, None] + torch.arange(S)[None, :])[:, :, None]
-    q[..., off:off + dims] = _rotate(q[..., off:off + dims].float(), pos, inv_freq, dims).to(q.dtype)
+    q[..., off:off + dims] = _rotate(q[..., off:off + dims].float(), pos, inv_freq, dims, amp).to(q.dtype)
     return q
 
 
@@ -259,14 +303,15 @@ LATENT_ROW_MAX = 640        # widest key-store row (latent + rotated part) the a
 
 
 def latent_window_attention(qa: torch.Tensor, q: torch.Tensor, off: int, keys: torch.Tensor, key_index: Optional[torch.Tensor],
-                            pos0: torch.Tensor, lens: torch.Tensor, window: int, scale: float) -> torch.Tensor:
+                            pos0: torch.Tensor, lens: torch.Tensor, window: int, scale: float, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``qa [H, B*S, C]`` absorbed queries, ``q [B,S,H,Dq]`` whose coordinates from ``off`` are the rotated part, ``keys
     [blocks, ring, C+R]`` (row ``j mod ring`` of block ``key_index[b]``, or of block b, holds position j).  Position p sees
-    ``p - window < j <= p``.  Returns the attention-weighted sum of the latents ``[H, B*S, C]``; padded rows give zeros."""
+    ``p - window < j <= p``; ``exp(sink[h])`` (``sink [H]`` float, optional) joins the softmax denominator.  Returns the
+    attention-weighted sum of the latents ``[H, B*S, C]``; padded rows give zeros."""
     if _cuda(qa):
         _ext.count_launch()
         return ext().latent_window_attention(qa, q, off, keys, None if key_index is None else _i32(key_index), _i32(pos0), _i32(lens),
-                                             window, scale)
+                                             window, scale, sink)
     H, N, C = qa.shape
     B, S = q.shape[:2]
     ring, R = keys.shape[1], keys.shape[2] - C
@@ -277,8 +322,10 @@ def latent_window_attention(qa: torch.Tensor, q: torch.Tensor, off: int, keys: t
     r = torch.arange(ring)
     j = p[..., None] - torch.remainder(p[..., None] - r, ring)                                       # position held by ring row r
     ok = (j >= 0) & (j > p[..., None] - window)
-    sc = sc.masked_fill(~ok[:, :, None, :], float("-inf"))
-    o = torch.einsum("bshr,brc->bshc", torch.softmax(sc, -1), kb.float()[..., :C])
+    live = ok.any(1)                                                                                 # rows no token of the step sees hold anything
+    kv = torch.where(live[..., None], kb.float()[..., :C], torch.zeros(()))
+    w = _sink_softmax(sc.permute(0, 2, 1, 3), sink, ok[:, None])                                     # [B,H,S,ring]
+    o = torch.einsum("bhsr,brc->bshc", w, kv)
     o = torch.where((torch.arange(S)[None, :] < lens[:, None])[..., None, None], o, torch.zeros_like(o))
     return o.permute(2, 0, 1, 3).reshape(H, N, C).to(qa.dtype)
 
@@ -289,23 +336,27 @@ def latent_prompt_fused_ok(q: torch.Tensor, D: int, R: int, CR: int, VD: int) ->
 
 
 def latent_prompt_attention(q: torch.Tensor, kx: torch.Tensor, rows: torch.Tensor, v: torch.Tensor, lens: torch.Tensor, D: int, R: int,
-                            VD: int, window: int, scale: float) -> torch.Tensor:
+                            VD: int, window: int, scale: float, sink: Optional[torch.Tensor] = None,
+                            gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Prompts that start at position 0, expanded form, one kernel (GPU, bfloat16): ``q [B,S,H,D+R]`` rotated queries, ``kx
     [B,S,H*D]`` every head's unrotated keys, ``rows [B,S,CR]`` whose last R numbers are the rotated key part all heads share, ``v
-    [B,S,H*VD]``.  Query i sees ``i - window < j <= i``.  Returns the heads' outputs ``[B*S, H*VD]``; padded rows give zeros."""
+    [B,S,H*VD]``.  Query i sees ``i - window < j <= i``; ``exp(sink[h])`` joins the denominator (optional).  Returns the heads' outputs
+    ``[B*S, H*VD]``, times ``sigmoid(gate [B*S, H*VD])`` (optional; row stride free); padded rows give zeros."""
     _ext.count_launch()
-    return ext().latent_prompt_attention(q, kx.contiguous(), rows, v.contiguous(), _i32(lens), D, R, VD, window, scale)
+    return ext().latent_prompt_attention(q, kx.contiguous(), rows, v.contiguous(), _i32(lens), D, R, VD, window, scale, sink, gate)
 
 
 def window_softmax(scores: torch.Tensor, scale: float, ring_mode: bool, H: int, Qb: int, nblk: int, w_eff: int, window: int,
-                   pos0: torch.Tensor, lens: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+                   pos0: torch.Tensor, lens: torch.Tensor, out_dtype: torch.dtype, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Softmax over the visible keys of float score rows made by block matrix products; masked entries come out as zeros.
     Band mode: ``scores [B, nblk, Qb*H, span]``, column kk of block ``blk`` is position ``blk*Qb - (w_eff-1) + kk``; the query of
     row ``(t, h)`` sits at ``i = blk*Qb + t`` and sees ``max(0, i-window+1) <= j <= i``; rows with ``i >= lens[b]`` are zeros.
-    Ring mode: ``scores [B, H, ring]`` of single tokens at ``pos0[b]``; ring row kk holds position ``p - ((p - kk) mod ring)``."""
+    Ring mode: ``scores [B, H, ring]`` of single tokens at ``pos0[b]``; ring row kk holds position ``p - ((p - kk) mod ring)``.
+    ``sink`` (float ``[n]``): ``exp`` of number ``(b * H + h) mod n`` joins the denominator of row ``(b, ..., h)``."""
     if _cuda(scores):
         _ext.count_launch()
-        return ext().window_softmax(scores, scale, ring_mode, H, Qb, nblk, w_eff, window, _i32(pos0), _i32(lens), out_dtype == torch.bfloat16)
+        return ext().window_softmax(scores, scale, ring_mode, H, Qb, nblk, w_eff, window, _i32(pos0), _i32(lens),
+                                    out_dtype == torch.bfloat16, sink)
     span = scores.shape[-1]
     kk = torch.arange(span)
     if ring_mode:
@@ -319,7 +370,13 @@ def window_softmax(scores: torch.Tensor, scale: float, ring_mode: bool, H: int, 
         ok = ok[None] & (i[None] < lens.long()[:, None, None, None])                                  # [B,nblk,Qb,span]
         ok = ok[:, :, :, None, :].expand(-1, -1, -1, H, -1).reshape(scores.shape)
     sc = (scores.float() * scale).masked_fill(~ok.expand(scores.shape), float("-inf"))
-    return torch.nan_to_num(torch.softmax(sc, -1), nan=0.0).to(out_dtype)
+    if sink is not None:
+        B = scores.shape[0]
+        row = sink[(torch.arange(B)[:, None] * H + torch.arange(H)[None, :]) % sink.numel()]          # [B,H]
+        row = row[:, :, None] if ring_mode else row[:, None, None, :].expand(B, nblk, Qb, H).reshape(B, nblk, Qb * H, 1)
+        sc = torch.cat([sc, row], -1)
+    p = torch.nan_to_num(torch.softmax(sc, -1), nan=0.0)[..., :span]
+    return p.to(out_dtype)
 
 
 SMALL_LINEAR_ROWS = 16        # up to this many rows a float-result product runs as one warp per output
@@ -340,25 +397,45 @@ ROUTE_MAX_EXPERTS = 256
 ROUTE_KINDS = {"sigmoid": 0, "softmax": 1, "softmax_top": 2}
 
 
-def route_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_real: int, act: str = "softmax", scale: float = 1.0):
+def route_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_real: int, act: str = "softmax", scale: float = 1.0,
+               groups=None, normalise: bool = False, gate_column: bool = False):
     """Float router logits ``[N, E]`` → ``(weights [N, top] float, expert ids [N, top] int64, identity share [N] float)``.
     ``scores = softmax / sigmoid(logits)``; the ``top`` largest of ``scores + correction`` are chosen (descending); a chosen expert
     below ``n_real`` gets weight ``score * scale``, a chosen expert from ``n_real`` on (an identity expert) gets weight 0 and adds its
     score to the row's identity share.  ``act="softmax_top"``: the ``top`` largest LOGITS are chosen and the weights are the softmax
-    over the chosen logits only (times ``scale``); no correction, no identity experts."""
-    if _cuda(logits) and logits.shape[1] <= ROUTE_MAX_EXPERTS:
+    over the chosen logits only (times ``scale``); no correction, no identity experts.  ``groups = (count, keep)``: the experts form
+    ``count`` equal groups of neighbours worth the sum of their two largest choice values each, and only experts of the ``keep`` best
+    groups can be chosen.  ``normalise``: the chosen scores are divided by their sum (+ 1e-20; no identity experts).
+    ``gate_column``: the logits have one more column, the logit of a gate, whose sigmoid is the third result."""
+    E = logits.shape[1] - (1 if gate_column else 0)
+    count, keep = groups if groups else (0, 0)
+    if count and (E % count or not 1 <= keep <= count or top > keep * (E // count)):
+        raise ValueError(f"{E} experts in {count} groups, {keep} kept, do not leave {top} to choose")
+    if normalise and n_real < E:
+        raise ValueError("identity experts with weights that sum to one")
+    if _cuda(logits) and E <= ROUTE_MAX_EXPERTS:
         _ext.count_launch()
-        w, idx, ident = ext().route_topk(logits.contiguous(), correction, top, n_real, ROUTE_KINDS[act], float(scale))
+        w, idx, ident = ext().route_topk(logits.contiguous(), correction, top, n_real, ROUTE_KINDS[act], float(scale), count, keep, normalise,
+                                         gate_column)
         return w, idx, ident
+    gate = torch.sigmoid(logits[:, E].float()) if gate_column else None
+    logits = logits[:, :E]
     if act == "softmax_top":
         val, idx = torch.topk(logits.float(), top, dim=-1)
-        return torch.softmax(val, -1) * scale, idx, torch.zeros(logits.shape[0], device=logits.device)
+        return torch.softmax(val, -1) * scale, idx, gate if gate_column else torch.zeros(logits.shape[0], device=logits.device)
     scores = torch.softmax(logits.float(), -1) if act == "softmax" else torch.sigmoid(logits.float())
-    idx = torch.topk(scores if correction is None else scores + correction, top, dim=-1).indices
+    choice = scores if correction is None else scores + correction
+    if count:
+        worth = choice.view(-1, count, E // count).topk(min(2, E // count), dim=-1).values.sum(-1)
+        kept = torch.zeros_like(worth, dtype=torch.bool).scatter_(1, worth.topk(keep, dim=-1).indices, True)
+        choice = choice.masked_fill(~kept.repeat_interleave(E // count, 1), float("-inf"))
+    idx = torch.topk(choice, top, dim=-1).indices
     w = scores.gather(1, idx)
+    if normalise:
+        w = w / (w.sum(1, keepdim=True) + 1e-20)
     real = idx < n_real
     ident = torch.where(real, torch.zeros_like(w), w).sum(1)
-    return torch.where(real, w * scale, torch.zeros_like(w)), idx, ident
+    return torch.where(real, w * scale, torch.zeros_like(w)), idx, gate if gate_column else ident
 
 
 def matmul_f32(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
@@ -786,6 +863,16 @@ def sigmoid_gate_mul_(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
     rep = C // gate.shape[1]
     x.copy_((x.float().view(N, -1, rep) * torch.sigmoid(gate.float())[..., None]).view(N, C).to(x.dtype))
     return x
+
+
+def sigmoid_gate_heads(ov: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """``ov [H, N, V]`` (heads as a batched product leaves them) times ``sigmoid(gate [N, H*V])`` (row stride free), packed to
+    ``[N, H*V]``."""
+    if _cuda(ov):
+        _ext.count_launch()
+        return ext().sigmoid_gate_heads(ov, gate)
+    H, N, V = ov.shape
+    return (ov.transpose(0, 1).reshape(N, H * V).float() * torch.sigmoid(gate.float())).to(ov.dtype)
 
 
 # ------------------------------------------------------------------------------------------------------- retention (fixed decay)
