@@ -175,9 +175,9 @@ latent_ring_partial_kernel(const T* __restrict__ qa, long qa_sn, long qa_sh, con
     }
 }
 
-// grid (H, B): merges the chunk partials of one (sequence, head) and writes out[h, b, :].  The chunks' weights exp(m_s - M) / L are
+// grid (H, B, column tiles): merges the chunk partials of one (sequence, head) and writes out[h, b, :].  The chunks' weights exp(m_s - M) / L are
 // formed once (a lane per chunk) and kept in shared memory; every thread then sums its columns over the chunks, loads unrolled.
-template <typename T>
+template <typename T, int VW>
 __global__ void latent_ring_merge_kernel(const float* __restrict__ part_m, const float* __restrict__ part_l,
                                          const float* __restrict__ part_acc, int nsplit, int H, int C, const float* __restrict__ sink,
                                          T* __restrict__ out, long out_sn, long out_sh) {
@@ -204,17 +204,35 @@ __global__ void latent_ring_merge_kernel(const float* __restrict__ part_m, const
     __syncthreads();
     T* o = out + (long)b * out_sn + (long)h * out_sh;
     if (red[0] == -INFINITY) {                 // a padded row: nothing visible anywhere
-        for (int c = tid; c < C; c += blockDim.x) stf(o + c, 0.f);
+        for (int c = blockIdx.z * blockDim.x + tid; c < C; c += gridDim.z * blockDim.x) stf(o + c, 0.f);
         return;
     }
     const float inv = 1.f / red[1];
-    for (int c = tid; c < C; c += blockDim.x) {
+    // eight chunks' sums in flight at once; chunks that saw nothing left none (what their room holds is not used)
+    for (int c = (blockIdx.z * blockDim.x + tid) * VW; c < C; c += gridDim.z * blockDim.x * VW) {
         const float* pa = part_acc + i0 * C + c;
-        float a = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < nsplit; ++s)
-            if (sw[s] > 0.f) a = fmaf(pa[(long)s * H * C], sw[s], a);      // chunks that saw nothing left no sums
-        stf(o + c, a * inv);
+        float a[VW];
+#pragma unroll
+        for (int e = 0; e < VW; ++e) a[e] = 0.f;
+        for (int s0 = 0; s0 < nsplit; s0 += 8) {
+            float w[8], any = 0.f;
+#pragma unroll
+            for (int u = 0; u < 8; ++u) { w[u] = s0 + u < nsplit ? sw[s0 + u] : 0.f; any += w[u]; }
+            if (any == 0.f) continue;
+            float v[8][VW];
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const float* src = pa + (long)min(s0 + u, nsplit - 1) * H * C;
+                if (VW == 4) *reinterpret_cast<float4*>(v[u]) = *reinterpret_cast<const float4*>(src);
+                else v[u][0] = src[0];
+            }
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+#pragma unroll
+                for (int e = 0; e < VW; ++e) a[e] = w[u] > 0.f ? fmaf(v[u][e], w[u], a[e]) : a[e];
+        }
+        if (VW == 4) st4(o + c, make_float4(a[0] * inv, a[1 % VW] * inv, a[2 % VW] * inv, a[3 % VW] * inv));
+        else stf(o + c, a[0] * inv);
     }
 }
 
@@ -248,10 +266,17 @@ static void ring_decode_launch(const void* qa, long qa_sn, long qa_sh, const voi
 template <typename T>
 static void ring_merge_launch(const float* part_m, const float* part_l, const float* part_acc, int nsplit, int B, int H, int C, const float* sink,
                               void* out, long out_sn, long out_sh, cudaStream_t s) {
-    const int mt = C >= 256 ? 256 : (C >= 128 ? 128 : 64);
     const size_t smem = nsplit * sizeof(float);
-    if (smem > 48 * 1024) cudaFuncSetAttribute(latent_ring_merge_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-    latent_ring_merge_kernel<T><<<dim3(H, B), mt, smem, s>>>(part_m, part_l, part_acc, nsplit, H, C, sink, (T*)out, out_sn, out_sh);
+    const bool vec = C % 4 == 0 && out_sn % 4 == 0 && out_sh % 4 == 0 && (uintptr_t)out % 16 == 0;
+    const int mt = 64, per = mt * (vec ? 4 : 1);
+    dim3 grid(H, B, (C + per - 1) / per);
+#define SEQMIX_MERGE(V)                                                                                                             \
+    do {                                                                                                                            \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(latent_ring_merge_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+        latent_ring_merge_kernel<T, V><<<grid, mt, smem, s>>>(part_m, part_l, part_acc, nsplit, H, C, sink, (T*)out, out_sn, out_sh); \
+    } while (0)
+    if (vec) SEQMIX_MERGE(4); else SEQMIX_MERGE(1);
+#undef SEQMIX_MERGE
 }
 
 void latent_ring_decode(const void* qa, int bf, long qa_sn, long qa_sh, const void* qr, long qr_sn, long qr_sh, const void* keys,

@@ -3,7 +3,8 @@
 // staged rows weighted are the value product over the C latent ones.
 // One block = one stretch of a sequence's visible positions x one tile of 16 heads.  The stretches divide what the token sees NOW
 // (position and window, read on the device), not the ring, so a long cache costs what the sequence has filled.  Rows arrive by
-// asynchronous copies, two tiles of 32 ahead of the arithmetic.  The eight warps split a tile's scores by (8 rows, half of the
+// asynchronous copies, a tile of 32 ahead of the arithmetic; two blocks share an SM, so one's copies and barriers run under the other's
+// arithmetic.  The eight warps split a tile's scores by (8 rows, half of the
 // coordinates); each then forms the softmax weights of all 16 x 32 pairs for itself (float; weights are rounded to bfloat16 only as
 // operands of the value product) and owns a share of the value columns, with float accumulators in registers.
 // A stretch leaves its maximum, sum of weights and unnormalised sums per head; latent_ring_merge_kernel (latent_decode.cu) folds them.
@@ -15,13 +16,13 @@ namespace seqmix {
 
 static const int kRows = 32;        // positions per tile
 static const int kHeadTile = 16;
-static const int kStages = 3;
+static const int kStages = 2;
 static const int kWarps = 8;
 static const int kScoreLd = kRows + 4;
 static const int kMaxRow = 640;     // C + R
 
 template <int NP>                   // pairs of 8-column value tiles per warp: C <= 16 * kWarps * NP
-__global__ void __launch_bounds__(32 * kWarps, 1)
+__global__ void __launch_bounds__(32 * kWarps, 2)
 latent_decode_mma_kernel(const bf16* __restrict__ qa, long qa_sn, long qa_sh, const bf16* __restrict__ qr, long qr_sn, long qr_sh,
                          const bf16* __restrict__ keys, long key_sb, int ring, const int* __restrict__ key_index,
                          const int* __restrict__ pos0, const int* __restrict__ lens, int H, int C, int R, int window, float scale2,
@@ -53,8 +54,6 @@ latent_decode_mma_kernel(const bf16* __restrict__ qa, long qa_sn, long qa_sh, co
     const int nt = (j1 - j0 + kRows - 1) / kRows;
     fetch(0);
     cp_commit();
-    if (nt > 1) fetch(1);
-    cp_commit();
     // the tile's queries: absorbed part, then rotated part; heads past the last are zeros
     for (int i = tid; i < kHeadTile * (C / 8); i += 32 * kWarps) {
         const int h = i / (C / 8), c = (i % (C / 8)) * 8;
@@ -73,9 +72,9 @@ latent_decode_mma_kernel(const bf16* __restrict__ qa, long qa_sn, long qa_sh, co
     for (int n = 0; n < 2 * NP; ++n) oacc[n][0] = oacc[n][1] = oacc[n][2] = oacc[n][3] = 0.f;
     float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
     for (int t = 0; t < nt; ++t) {
-        cp_wait<1>();
+        cp_wait<0>();
         __syncthreads();                                   // tile t (and the queries) are here; everyone has left tile t - 1
-        if (t + 2 < nt) fetch(t + 2);
+        if (t + 1 < nt) fetch(t + 1);
         cp_commit();
         const bf16* Kt = Ks + (t % kStages) * kRows * ld;
         float sacc[4] = {0.f, 0.f, 0.f, 0.f}, sacd[4] = {0.f, 0.f, 0.f, 0.f};
@@ -175,9 +174,9 @@ latent_decode_mma_kernel(const bf16* __restrict__ qa, long qa_sn, long qa_sh, co
 
 bool latent_decode_mma_fits(int C, int R) { return C % 16 == 0 && R % 16 == 0 && C > 0 && C + R <= kMaxRow; }
 
-// enough stretches to give every SM a block, but none shorter than a tile
+// as many stretches as fill the GPU once (two blocks per SM), but none shorter than a tile
 int latent_decode_mma_splits(int B, int H, int rows) {
-    const int units = B * ((H + kHeadTile - 1) / kHeadTile), want = (148 + units - 1) / units, most = (rows + kRows - 1) / kRows;
+    const int units = B * ((H + kHeadTile - 1) / kHeadTile), want = 2 * 148 / units, most = (rows + kRows - 1) / kRows;
     return want < 1 ? 1 : (want < most ? want : (most < 1 ? 1 : most));
 }
 
