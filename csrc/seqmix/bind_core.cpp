@@ -219,12 +219,12 @@ void group_rms_norm_gated(const Tensor& x, const Tensor& gate, const Tensor& w, 
 // kind 1: softmax, 0: sigmoid, 2: softmax over the chosen; groups / gkeep: the choice is limited to the best groups; norm: weights sum to 1
 std::vector<Tensor> route_topk(const Tensor& logits, const c10::optional<Tensor>& correction, int64_t top, int64_t n_real, int64_t kind,
                                double scale, int64_t groups, int64_t gkeep, bool norm, bool share) {
-    TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.is_contiguous() && logits.scalar_type() == at::kFloat, "logits must be float [N,E]");
+    TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1 && logits.scalar_type() == at::kFloat, "logits must be float [N,E]");
     const int N = logits.size(0), E = logits.size(1) - (share ? 1 : 0);
     TORCH_CHECK(!correction || correction->numel() == E, "the correction holds one number per expert");
     Tensor w = at::empty({N, top}, logits.options()), idx = at::empty({N, top}, logits.options().dtype(at::kLong));
     Tensor ident = at::empty({N}, logits.options());
-    bool ok = seqmix::route_topk(logits.data_ptr<float>(), logits.size(1), correction ? f32(*correction) : nullptr, N, E, (int)top, (int)n_real, (int)kind,
+    bool ok = seqmix::route_topk(logits.data_ptr<float>(), logits.stride(0), correction ? f32(*correction) : nullptr, N, E, (int)top, (int)n_real, (int)kind,
                                  (float)scale, (int)groups, (int)gkeep, norm, share, w.data_ptr<float>(), idx.data_ptr<int64_t>(), ident.data_ptr<float>(), stream());
     TORCH_CHECK(ok, "route_topk: at most 256 experts, top <= experts, equal groups that leave enough to choose from");
     check_launch();

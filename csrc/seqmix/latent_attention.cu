@@ -97,49 +97,53 @@ __global__ void latent_kv_store_vec_kernel(const T* __restrict__ kv, long kv_sb,
     const T* x = kv + (long)b * kv_sb + (long)t * kv_st;
     T* dst_row = rows ? rows + (long)n * CR : nullptr;
     T* dst_cache = (cache && t >= len - ring) ? cache + ((long)slots[b] * ring + (p % ring)) * CR : nullptr;
+    const bool kv_part = blockIdx.y == 0;       // gridDim.y > 1 (few tokens): the query heads go to blocks of their own
     float4 v[kStoreVec];
     float ss = 0.f;
+    if (kv_part) {
 #pragma unroll
-    for (int e = 0; e < kStoreVec; ++e) {
-        const int c = (e * 32 + lane) * 4;
-        v[e] = c < C ? ld4(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        ss = fmaf(v[e].x, v[e].x, fmaf(v[e].y, v[e].y, fmaf(v[e].z, v[e].z, fmaf(v[e].w, v[e].w, ss))));
-    }
-    ss = warp_sum(ss);
-    const float inv = 1.f / sqrtf(ss / (float)C + eps);
+        for (int e = 0; e < kStoreVec; ++e) {
+            const int c = (e * 32 + lane) * 4;
+            v[e] = c < C ? ld4(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss = fmaf(v[e].x, v[e].x, fmaf(v[e].y, v[e].y, fmaf(v[e].z, v[e].z, fmaf(v[e].w, v[e].w, ss))));
+        }
+        ss = warp_sum(ss);
+        const float inv = 1.f / sqrtf(ss / (float)C + eps);
 #pragma unroll
-    for (int e = 0; e < kStoreVec; ++e) {
-        const int c = (e * 32 + lane) * 4;
-        if (c < C) {
-            const float4 g = ld4(nw + c);
-            const float4 o = make_float4(v[e].x * inv * g.x, v[e].y * inv * g.y, v[e].z * inv * g.z, v[e].w * inv * g.w);
-            if (dst_row) st4(dst_row + c, o);
-            if (dst_cache) st4(dst_cache + c, o);
+        for (int e = 0; e < kStoreVec; ++e) {
+            const int c = (e * 32 + lane) * 4;
+            if (c < C) {
+                const float4 g = ld4(nw + c);
+                const float4 o = make_float4(v[e].x * inv * g.x, v[e].y * inv * g.y, v[e].z * inv * g.z, v[e].w * inv * g.w);
+                if (dst_row) st4(dst_row + c, o);
+                if (dst_cache) st4(dst_cache + c, o);
+            }
+        }
+        for (int i = lane * 4; i < half; i += 128) {
+            const float4 u = ld4(x + C + i), w = ld4(x + C + i + half), f = ld4(inv_freq + i);
+            float4 sn, cs;
+            sincosf((float)p * f.x, &sn.x, &cs.x); sincosf((float)p * f.y, &sn.y, &cs.y);
+            sincosf((float)p * f.z, &sn.z, &cs.z); sincosf((float)p * f.w, &sn.w, &cs.w);
+            scale4(sn, amp); scale4(cs, amp);
+            const float4 a = turn_lo(u, w, sn, cs), bb = turn_hi(u, w, sn, cs);
+            if (dst_row) { st4(dst_row + C + i, a); st4(dst_row + C + i + half, bb); }
+            if (dst_cache) { st4(dst_cache + C + i, a); st4(dst_cache + C + i + half, bb); }
+        }
+        for (int i = dims + lane; i < R; i += 32) {      // coordinates past the rotated ones pass unchanged
+            float u = ldf(x + C + i);
+            if (dst_row) stf(dst_row + C + i, u);
+            if (dst_cache) stf(dst_cache + C + i, u);
         }
     }
-    for (int i = lane * 4; i < half; i += 128) {
-        const float4 u = ld4(x + C + i), w = ld4(x + C + i + half), f = ld4(inv_freq + i);
-        float4 sn, cs;
-        sincosf((float)p * f.x, &sn.x, &cs.x); sincosf((float)p * f.y, &sn.y, &cs.y);
-        sincosf((float)p * f.z, &sn.z, &cs.z); sincosf((float)p * f.w, &sn.w, &cs.w);
-        scale4(sn, amp); scale4(cs, amp);
-        const float4 a = turn_lo(u, w, sn, cs), bb = turn_hi(u, w, sn, cs);
-        if (dst_row) { st4(dst_row + C + i, a); st4(dst_row + C + i + half, bb); }
-        if (dst_cache) { st4(dst_cache + C + i, a); st4(dst_cache + C + i + half, bb); }
-    }
-    for (int i = dims + lane; i < R; i += 32) {      // coordinates past the rotated ones pass unchanged
-        float u = ldf(x + C + i);
-        if (dst_row) stf(dst_row + C + i, u);
-        if (dst_cache) stf(dst_cache + C + i, u);
-    }
-    if (q && dims > 0) {
+    if (q && dims > 0 && (gridDim.y == 1 || !kv_part)) {
         const int quads = dims / 8, i = (lane % quads) * 4;
         const float4 f = ld4(inv_freq + i);
         float4 sn, cs;
         sincosf((float)p * f.x, &sn.x, &cs.x); sincosf((float)p * f.y, &sn.y, &cs.y);
         sincosf((float)p * f.z, &sn.z, &cs.z); sincosf((float)p * f.w, &sn.w, &cs.w);
         scale4(sn, amp); scale4(cs, amp);
-        for (int h = lane / quads; h < H; h += 32 / quads) {
+        const int step = 32 / quads, turn = gridDim.y > 1 ? blockIdx.y - 1 : 0, turns = gridDim.y > 1 ? gridDim.y - 1 : 1;
+        for (int h = turn * step + lane / quads; h < H; h += turns * step) {
             T* y = q + (long)n * q_sn + (long)h * q_sh + i;
             const float4 u = ld4(y), w = ld4(y + half);
             st4(y, turn_lo(u, w, sn, cs));
@@ -283,6 +287,7 @@ void latent_kv_store(const void* kv, int bf, long kv_sb, long kv_st, int B, int 
     const bool with_q = vec && q && dims > 0 && 32 % (dims / 8) == 0 && q_sn % 4 == 0 && q_sh % 4 == 0 && al(q);
     if (q && !with_q) rope_q(q, bf, q_sn, q_sh, B * S, S, H, dims, inv_freq, pos0, amp, s);
     void* qf = with_q ? q : nullptr;
+    if (with_q && B * S <= 256) grid.y = 1 + (H + 32 / (dims / 8) - 1) / (32 / (dims / 8));
     if (vec) {
         if (bf) latent_kv_store_vec_kernel<bf16><<<grid, block, 0, s>>>((const bf16*)kv, kv_sb, kv_st, B, S, C, R, dims, nw, eps, inv_freq, pos0,
                                                                        lens, slots, (bf16*)cache, ring, (bf16*)rows, amp, (bf16*)qf, q_sn, q_sh, H);

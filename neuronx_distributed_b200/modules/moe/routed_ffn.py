@@ -79,10 +79,12 @@ class RoutedFFN(nn.Module):
             return F.linear(h.float(), w)
         if self._router_lowp is None or self._router_lowp[0] != w._version:
             low = w.detach().to(torch.bfloat16)
-            self._router_lowp = (w._version, low.t().contiguous() if bool((low.float() == w).all()) else None)
+            fits = bool((low.float() == w).all())
+            pad = F.pad(low, (0, 0, 0, -w.shape[0] % 8))               # whole 16 bytes of outputs: the aligned matrix products take it
+            self._router_lowp = (w._version, pad.t().contiguous() if fits else None)
         if self._router_lowp[1] is None:
             return F.linear(h.float(), w)
-        return seqmix.matmul_f32(h[None], self._router_lowp[1][None])[0]
+        return seqmix.matmul_f32(h[None], self._router_lowp[1][None])[0][:, :w.shape[0]]
 
     def route(self, h: torch.Tensor):
         """Float scores of all experts → (weights ``[N, top]`` float, expert ids ``[N, top]``, identity share or shared expert's gate

@@ -415,7 +415,7 @@ def route_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: in
         raise ValueError("identity experts with weights that sum to one")
     if _cuda(logits) and E <= ROUTE_MAX_EXPERTS:
         _ext.count_launch()
-        w, idx, ident = ext().route_topk(logits.contiguous(), correction, top, n_real, ROUTE_KINDS[act], float(scale), count, keep, normalise,
+        w, idx, ident = ext().route_topk(logits if logits.stride(1) == 1 else logits.contiguous(), correction, top, n_real, ROUTE_KINDS[act], float(scale), count, keep, normalise,
                                          gate_column)
         return w, idx, ident
     gate = torch.sigmoid(logits[:, E].float()) if gate_column else None

@@ -276,6 +276,20 @@ def test_attention_prompt_and_cache(device, H, D, R, V, C, S, order):
 
 
 @pytest.mark.parametrize("device", DEVICES)
+def test_rows_wider_than_the_single_token_kernels_take(device):
+    """Latents beyond the decode kernels' row limit go through matrix products over the cache."""
+    H, D, R, V, C, S = 2, 8, 8, 8, seqmix.LATENT_ROW_MAX, 14
+    cfg, w, h, want = _attention_case(H, D, R, V, C, S, 77)
+    mix = build(cfg, w, device, max_seq_len=S + 2).lm.layers[0].mixer
+    st = {"kv": torch.full((2, S + 2, C + R), 9.0, device=device)}
+    tol = 2e-4 * max(1.0, want.abs().max().item())
+    for cut in (5, S):
+        out = [mix(h[:cut].to(device)[None], _Ctx([cut], [1], [0], True, device), st)[0]]
+        out += [mix(h[t:t + 1].to(device)[None], _Ctx([1], [1], [t], False, device), st)[0] for t in range(cut, S)]
+        assert (torch.cat(out).cpu().double() - want).abs().max() < tol
+
+
+@pytest.mark.parametrize("device", DEVICES)
 def test_absorbed_attention_takes_part_in_no_row_it_does_not_see(device):
     """Cache rows never written hold NaN here: they may not reach any result."""
     H, C, R, ring = 3, 20, 6, 50
