@@ -3,13 +3,15 @@
 //   gelu_erf     : 0.5 z (1 + erf(z / sqrt 2))
 //   relu_sq      : max(z, 0)^2
 //   silu_mul     : silu(gate) * up for rows [gate | up]
-//   clamped_glu  : g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(slope g) (u + 1) for rows [gate | up]
+//   clamped_glu  : g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(slope g) (u + 1) for rows [gate | up]; a number per row
+//                  may multiply both first (an expert that reads weight * h: the products are linear, so the weight enters here)
 //   sigmoid_gate_mul : x *= sigmoid(gate), one gate number per `rep` consecutive coordinates (a head, or one coordinate)
 //   indexed_gemv : out[m,:] = act(W[sel[m]] x[m,:]) for a few rows m, each with its own matrix out of a stack [E, O, I]
 //                  (token generation: the chosen experts' matrices are streamed once, a warp per output row); act 0: none,
 //                  1: gelu_erf, 2: the matrix stacks gate rows over up rows and out = silu(gate row . x) * (up row . x), O/2 columns;
-//                  3: the square of relu; rows whose sel names no matrix give zeros
-//   moe_combine  : y[n,:] = base_weight[n] * base[n,:] + sum_k weight[n,k] * rows[src[n,k],:], summed in float
+//                  3: the square of relu; 4: like 2 with the activation of clamped_glu; a number per row may multiply x[m,:] (in
+//                  float, on the products); rows whose sel names no matrix give zeros
+//   moe_combine  : y[n,:] = base_weight[n] * base[n,:] + sum_k weight[n,k] * rows[src[n,k],:], summed in float (no weights: ones)
 //   route_topk   : scores, choice with a correction (optionally only among the best groups of neighbouring experts), top-k, weights
 //                  (optionally divided by their sum) and the identity experts' share or the shared expert's gate in one launch
 //   sigmoid_gate_heads : heads laid out [H, N, V] times sigmoid of a gate per coordinate, packed to [N, H * V]
@@ -82,10 +84,17 @@ __device__ __forceinline__ float row_dot(const T* __restrict__ wr, const T* __re
     return warp_sum(acc);
 }
 
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float slope) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoidf_(slope * g) * (u + 1.f);
+}
+
 template <typename T, bool VEC>
 __global__ void indexed_gemv_kernel(const T* __restrict__ w, const int* __restrict__ sel, const T* __restrict__ x, long x_stride,
-                                    int M, int E, int O, int I, int act, T* __restrict__ out) {
-    const int On = act == 2 ? O / 2 : O;
+                                    const float* __restrict__ x_scale, int M, int E, int O, int I, int act, float limit, float slope,
+                                    T* __restrict__ out) {
+    const int On = (act == 2 || act == 4) ? O / 2 : O;
     const int o = blockIdx.x * blockDim.y + threadIdx.y, m = blockIdx.y, lane = threadIdx.x;
     if (o >= On) return;
     const int e = sel[m];
@@ -95,10 +104,12 @@ __global__ void indexed_gemv_kernel(const T* __restrict__ w, const int* __restri
     }
     const T* wr = w + ((long)e * O + o) * I;
     const T* xr = x + (long)m * x_stride;
-    float acc = row_dot<T, VEC>(wr, xr, I, lane);
+    const float xs = x_scale ? x_scale[m] : 1.f;
+    float acc = row_dot<T, VEC>(wr, xr, I, lane) * xs;
     if (act == 1) acc = gelu_erf_(acc);
     else if (act == 3) acc = relu_sq_(acc);
-    else if (act == 2) acc = acc * sigmoidf_(acc) * row_dot<T, VEC>(wr + (long)On * I, xr, I, lane);
+    else if (act == 2) acc = acc * sigmoidf_(acc) * (row_dot<T, VEC>(wr + (long)On * I, xr, I, lane) * xs);
+    else if (act == 4) acc = clamped_glu_f(acc, row_dot<T, VEC>(wr + (long)On * I, xr, I, lane) * xs, limit, slope);
     if (lane == 0) stf(out + (long)m * On + o, acc);
 }
 
@@ -119,7 +130,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, const int* __rest
     const int c = blockIdx.x * blockDim.x + threadIdx.x, n = blockIdx.y;
     if (c >= C) return;
     float acc = base ? ldf(base + (long)n * C + c) * (base_weight ? base_weight[n] : 1.f) : 0.f;
-    for (int k = 0; k < top; ++k) acc = fmaf(weight[(long)n * top + k], ldf(rows + (long)src[(long)n * top + k] * C + c), acc);
+    for (int k = 0; k < top; ++k) acc = fmaf(weight ? weight[(long)n * top + k] : 1.f, ldf(rows + (long)src[(long)n * top + k] * C + c), acc);
     stf(out + (long)n * C + c, acc);
 }
 
@@ -331,39 +342,34 @@ void silu_mul(const void* gu, void* out, int bf, long rows, int F, cudaStream_t 
     else silu_mul_kernel<float><<<blocks, 256, 0, s>>>((const float*)gu, rows, F, (float*)out);
 }
 
-__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float slope) {
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return g * sigmoidf_(slope * g) * (u + 1.f);
-}
-
 template <typename T, bool VEC>
-__global__ void clamped_glu_kernel(const T* __restrict__ gu, long rows, int F, float limit, float slope, T* __restrict__ out) {
+__global__ void clamped_glu_kernel(const T* __restrict__ gu, const float* __restrict__ row_scale, long rows, int F, float limit, float slope, T* __restrict__ out) {
     const long i = ((long)blockIdx.x * blockDim.x + threadIdx.x) * (VEC ? 4 : 1);
     if (i >= rows * F) return;
     const long r = i / F;
     const int c = (int)(i - r * F);
+    const float w = row_scale ? row_scale[r] : 1.f;
     if (VEC) {
         const float4 g = ld4(gu + r * 2 * F + c), u = ld4(gu + r * 2 * F + F + c);
-        st4(out + i, make_float4(clamped_glu_f(g.x, u.x, limit, slope), clamped_glu_f(g.y, u.y, limit, slope),
-                                 clamped_glu_f(g.z, u.z, limit, slope), clamped_glu_f(g.w, u.w, limit, slope)));
+        st4(out + i, make_float4(clamped_glu_f(w * g.x, w * u.x, limit, slope), clamped_glu_f(w * g.y, w * u.y, limit, slope),
+                                 clamped_glu_f(w * g.z, w * u.z, limit, slope), clamped_glu_f(w * g.w, w * u.w, limit, slope)));
     } else {
-        stf(out + i, clamped_glu_f(ldf(gu + r * 2 * F + c), ldf(gu + r * 2 * F + F + c), limit, slope));
+        stf(out + i, clamped_glu_f(w * ldf(gu + r * 2 * F + c), w * ldf(gu + r * 2 * F + F + c), limit, slope));
     }
 }
 
-void clamped_glu(const void* gu, void* out, int bf, long rows, int F, float limit, float slope, cudaStream_t s) {
+void clamped_glu(const void* gu, const float* row_scale, void* out, int bf, long rows, int F, float limit, float slope, cudaStream_t s) {
     if (rows * F == 0) return;
     const size_t a4 = bf ? 8 : 16;
     if (F % 4 == 0 && (uintptr_t)gu % a4 == 0 && (uintptr_t)out % a4 == 0) {
         const unsigned vblocks = (unsigned)((rows * F / 4 + 255) / 256);
-        if (bf) clamped_glu_kernel<bf16, true><<<vblocks, 256, 0, s>>>((const bf16*)gu, rows, F, limit, slope, (bf16*)out);
-        else clamped_glu_kernel<float, true><<<vblocks, 256, 0, s>>>((const float*)gu, rows, F, limit, slope, (float*)out);
+        if (bf) clamped_glu_kernel<bf16, true><<<vblocks, 256, 0, s>>>((const bf16*)gu, row_scale, rows, F, limit, slope, (bf16*)out);
+        else clamped_glu_kernel<float, true><<<vblocks, 256, 0, s>>>((const float*)gu, row_scale, rows, F, limit, slope, (float*)out);
         return;
     }
     const unsigned blocks = (unsigned)((rows * F + 255) / 256);
-    if (bf) clamped_glu_kernel<bf16, false><<<blocks, 256, 0, s>>>((const bf16*)gu, rows, F, limit, slope, (bf16*)out);
-    else clamped_glu_kernel<float, false><<<blocks, 256, 0, s>>>((const float*)gu, rows, F, limit, slope, (float*)out);
+    if (bf) clamped_glu_kernel<bf16, false><<<blocks, 256, 0, s>>>((const bf16*)gu, row_scale, rows, F, limit, slope, (bf16*)out);
+    else clamped_glu_kernel<float, false><<<blocks, 256, 0, s>>>((const float*)gu, row_scale, rows, F, limit, slope, (float*)out);
 }
 
 // x [rows, C] contiguous, gate [rows, C / rep] with its own row stride
@@ -452,14 +458,14 @@ void sigmoid_gate_heads(const void* ov, const void* gate, long gate_stride, int 
 #undef SEQMIX_SGH
 }
 
-void indexed_gemv(const void* w, const int* sel, const void* x, int bf, long x_stride, int M, int E, int O, int I, int act, void* out,
-                  cudaStream_t s) {
+void indexed_gemv(const void* w, const int* sel, const void* x, int bf, long x_stride, const float* x_scale, int M, int E, int O, int I, int act,
+                  float limit, float slope, void* out, cudaStream_t s) {
     if (M == 0) return;
-    const int On = act == 2 ? O / 2 : O;
+    const int On = (act == 2 || act == 4) ? O / 2 : O;
     dim3 block(32, 8), grid((On + 7) / 8, M);
     const size_t a4 = bf ? 8 : 16;
     const bool vec = I % 4 == 0 && x_stride % 4 == 0 && (uintptr_t)w % a4 == 0 && (uintptr_t)x % a4 == 0;
-#define SEQMIX_IGEMV(T, V) indexed_gemv_kernel<T, V><<<grid, block, 0, s>>>((const T*)w, sel, (const T*)x, x_stride, M, E, O, I, act, (T*)out)
+#define SEQMIX_IGEMV(T, V) indexed_gemv_kernel<T, V><<<grid, block, 0, s>>>((const T*)w, sel, (const T*)x, x_stride, x_scale, M, E, O, I, act, limit, slope, (T*)out)
     if (bf) { if (vec) SEQMIX_IGEMV(bf16, true); else SEQMIX_IGEMV(bf16, false); }
     else { if (vec) SEQMIX_IGEMV(float, true); else SEQMIX_IGEMV(float, false); }
 #undef SEQMIX_IGEMV
@@ -475,7 +481,7 @@ __global__ void moe_combine_vec_kernel(const T* __restrict__ rows, const int* __
     float4 acc = base ? ld4(base + (long)n * C + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     if (base && base_weight) { const float bw = base_weight[n]; acc.x *= bw; acc.y *= bw; acc.z *= bw; acc.w *= bw; }
     for (int k = 0; k < top; ++k) {
-        const float w = weight[(long)n * top + k];
+        const float w = weight ? weight[(long)n * top + k] : 1.f;
         const float4 r = ld4(rows + (long)src[(long)n * top + k] * C + c);
         acc.x = fmaf(w, r.x, acc.x); acc.y = fmaf(w, r.y, acc.y); acc.z = fmaf(w, r.z, acc.z); acc.w = fmaf(w, r.w, acc.w);
     }

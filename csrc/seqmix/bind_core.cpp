@@ -76,12 +76,15 @@ Tensor relu_sq(const Tensor& x) {
 }
 
 // w [E,O,I], sel int [M], x [M,I] → act(w[sel[m]] x[m]): [M,O], or [M,O/2] for the gated kind (act 2)
-Tensor indexed_gemv(const Tensor& w, const Tensor& sel, const Tensor& x, int64_t act) {
+Tensor indexed_gemv(const Tensor& w, const Tensor& sel, const Tensor& x, int64_t act, const c10::optional<Tensor>& x_scale, double limit,
+                    double slope) {
     TORCH_CHECK(w.is_cuda() && w.dim() == 3 && w.is_contiguous() && x.dim() == 2 && x.stride(1) == 1 && x.scalar_type() == w.scalar_type(), "bad gemv operands");
     const int M = x.size(0), E = w.size(0), O = w.size(1), I = w.size(2);
-    TORCH_CHECK(x.size(1) == I && sel.numel() == M && act >= 0 && act <= 3 && (act != 2 || O % 2 == 0), "shape mismatch");
-    Tensor out = at::empty({M, act == 2 ? O / 2 : O}, x.options());
-    seqmix::indexed_gemv(w.data_ptr(), i32(sel), x.data_ptr(), is_bf(x), x.stride(0), M, E, O, I, (int)act, out.data_ptr(), stream());
+    const bool glu = act == 2 || act == 4;
+    TORCH_CHECK(x.size(1) == I && sel.numel() == M && act >= 0 && act <= 4 && (!glu || O % 2 == 0) && (!x_scale || x_scale->numel() == M), "shape mismatch");
+    Tensor out = at::empty({M, glu ? O / 2 : O}, x.options());
+    seqmix::indexed_gemv(w.data_ptr(), i32(sel), x.data_ptr(), is_bf(x), x.stride(0), x_scale ? f32(*x_scale) : nullptr, M, E, O, I, (int)act,
+                         (float)limit, (float)slope, out.data_ptr(), stream());
     check_launch();
     return out;
 }
@@ -95,15 +98,15 @@ Tensor silu_mul(const Tensor& gu) {
     return out;
 }
 
-// rows [M,C], src int [N,top], weight float [N,top], base [N,C] or none (times base_weight float [N] if given) → [N,C]
-Tensor moe_combine(const Tensor& rows, const Tensor& src, const Tensor& weight, const c10::optional<Tensor>& base,
+// rows [M,C], src int [N,top], weight float [N,top] (or none: ones), base [N,C] or none (times base_weight float [N] if given) → [N,C]
+Tensor moe_combine(const Tensor& rows, const Tensor& src, const c10::optional<Tensor>& weight, const c10::optional<Tensor>& base,
                    const c10::optional<Tensor>& base_weight) {
     TORCH_CHECK(rows.is_cuda() && rows.dim() == 2 && rows.is_contiguous() && src.dim() == 2, "bad combine operands");
     const int N = src.size(0), top = src.size(1), C = rows.size(1);
     if (base) TORCH_CHECK(base->is_contiguous() && base->scalar_type() == rows.scalar_type() && base->size(0) == N && base->size(1) == C, "bad base");
     if (base_weight) TORCH_CHECK(base && base_weight->numel() == N, "base_weight needs a base and one number per row");
     Tensor out = at::empty({N, C}, rows.options());
-    seqmix::moe_combine(rows.data_ptr(), i32(src), f32(weight), base ? base->data_ptr() : nullptr, base_weight ? f32(*base_weight) : nullptr,
+    seqmix::moe_combine(rows.data_ptr(), i32(src), weight ? f32(*weight) : nullptr, base ? base->data_ptr() : nullptr, base_weight ? f32(*base_weight) : nullptr,
                         is_bf(rows), N, top, C, out.data_ptr(), stream());
     check_launch();
     return out;
@@ -166,29 +169,40 @@ void postnorm_gated_(Tensor x, const Tensor& y, const c10::optional<Tensor>& gat
 
 // x float [rows, C] (in place) += scale * y, then h = norm(x) * w + bias of y's dtype (undefined tensor without w).  y: [rows, C], or with
 // src / weight [rows, top] the contiguous expert rows [M, C] of a routed feed-forward (base [rows, C] times base_weight [rows] added).
-Tensor residual_norm_(Tensor x, const Tensor& y, const c10::optional<Tensor>& scale, const c10::optional<Tensor>& w,
-                      const c10::optional<Tensor>& bias, double eps, bool center, const c10::optional<Tensor>& src,
-                      const c10::optional<Tensor>& weight, const c10::optional<Tensor>& base, const c10::optional<Tensor>& base_weight) {
-    TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.stride(1) == 1 && x.scalar_type() == at::kFloat && y.dim() == 2 && y.stride(1) == 1 &&
-                    y.size(1) == x.size(1), "x must be float [rows, C], y rows of C numbers");
+// y may be absent (nothing is added then) and `like` names h's dtype.  w2: a second gain, its result comes second.  inj_rows int64 [rows] and
+// inj_table [*, C] of h's dtype: a table row per row of x joins the sum; inj_vec float [C] as well.
+std::vector<Tensor> residual_norm_(Tensor x, const c10::optional<Tensor>& y, const c10::optional<Tensor>& scale, const c10::optional<Tensor>& w,
+                                   const c10::optional<Tensor>& bias, double eps, bool center, const c10::optional<Tensor>& src,
+                                   const c10::optional<Tensor>& weight, const c10::optional<Tensor>& base, const c10::optional<Tensor>& base_weight,
+                                   const c10::optional<Tensor>& w2, const c10::optional<Tensor>& inj_rows, const c10::optional<Tensor>& inj_table,
+                                   const c10::optional<Tensor>& inj_vec, const Tensor& like) {
+    TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.stride(1) == 1 && x.scalar_type() == at::kFloat, "x must be float [rows, C]");
     const int rows = x.size(0), C = x.size(1);
-    for (auto* t : {&scale, &w, &bias}) TORCH_CHECK(!*t || (*t)->numel() == C, "scale, weight and bias hold C numbers");
+    if (y) TORCH_CHECK(y->dim() == 2 && y->stride(1) == 1 && y->size(1) == C && y->scalar_type() == like.scalar_type(), "y must hold rows of C numbers");
+    for (auto* t : {&scale, &w, &bias, &w2, &inj_vec}) TORCH_CHECK(!*t || (*t)->numel() == C, "scale, weights, bias and vector hold C numbers");
+    TORCH_CHECK(!w2 || (w && !bias), "a second gain goes with a first one and without a bias");
     int top = 0;
     if (src) {
-        TORCH_CHECK(weight && src->dim() == 2 && src->size(0) == rows && weight->sizes() == src->sizes() && y.is_contiguous(), "bad expert operands");
+        TORCH_CHECK(y && src->dim() == 2 && src->size(0) == rows && (!weight || weight->sizes() == src->sizes()) && y->is_contiguous(), "bad expert operands");
         top = src->size(1);
     } else {
-        TORCH_CHECK(y.size(0) == rows && !base, "one row of y per row of x");
+        TORCH_CHECK((!y || y->size(0) == rows) && !base && !weight, "one row of y per row of x");
     }
-    if (base) TORCH_CHECK(base->is_contiguous() && base->scalar_type() == y.scalar_type() && base->size(0) == rows && base->size(1) == C, "bad base");
+    if (base) TORCH_CHECK(base->is_contiguous() && base->scalar_type() == like.scalar_type() && base->size(0) == rows && base->size(1) == C, "bad base");
     if (base_weight) TORCH_CHECK(base && base_weight->numel() == rows, "base_weight needs a base and one number per row");
-    Tensor h = w ? at::empty({rows, C}, y.options()) : Tensor();
-    seqmix::residual_norm(x.data_ptr<float>(), x.stride(0), y.data_ptr(), y.stride(0), is_bf(y), src ? i32(*src) : nullptr,
+    TORCH_CHECK(inj_rows.has_value() == inj_table.has_value(), "a table comes with the rows to take");
+    if (inj_rows) TORCH_CHECK(inj_rows->is_cuda() && inj_rows->is_contiguous() && inj_rows->scalar_type() == at::kLong && inj_rows->numel() == rows &&
+                                  inj_table->is_contiguous() && inj_table->dim() == 2 && inj_table->size(1) == C && inj_table->size(0) > 0 &&
+                                  inj_table->scalar_type() == like.scalar_type(), "bad table operands");
+    Tensor h = w ? at::empty({rows, C}, like.options()) : Tensor(), h2 = w2 ? at::empty({rows, C}, like.options()) : Tensor();
+    seqmix::residual_norm(x.data_ptr<float>(), x.stride(0), y ? y->data_ptr() : nullptr, y ? y->stride(0) : C, is_bf(like), src ? i32(*src) : nullptr,
                           weight ? f32(*weight) : nullptr, top, base ? base->data_ptr() : nullptr, base_weight ? f32(*base_weight) : nullptr,
                           scale ? f32(*scale) : nullptr, w ? f32(*w) : nullptr, bias ? f32(*bias) : nullptr, (float)eps, center, rows, C,
-                          w ? h.data_ptr() : nullptr, C, stream());
+                          w ? h.data_ptr() : nullptr, C, w2 ? f32(*w2) : nullptr, w2 ? h2.data_ptr() : nullptr,
+                          inj_rows ? inj_rows->data_ptr<int64_t>() : nullptr, inj_table ? inj_table->data_ptr() : nullptr,
+                          inj_table ? (int)inj_table->size(0) : 0, inj_vec ? f32(*inj_vec) : nullptr, stream());
     check_launch();
-    return h;
+    return {h, h2};
 }
 
 // ov [H, N, V] contiguous, gate [N, H * V] of its dtype (row stride free) → [N, H * V] = heads packed, times sigmoid(gate)
@@ -242,10 +256,11 @@ Tensor small_linear_f32(const Tensor& x, const Tensor& w) {
 }
 
 // gu [M, 2F] contiguous → g sigmoid(slope g) (u + 1) with g = min(gu[:, :F], limit), u = clamp(gu[:, F:], -limit, limit)
-Tensor clamped_glu(const Tensor& gu, double limit, double slope) {
+Tensor clamped_glu(const Tensor& gu, double limit, double slope, const c10::optional<Tensor>& row_scale) {
     TORCH_CHECK(gu.is_cuda() && gu.dim() == 2 && gu.is_contiguous() && gu.size(1) % 2 == 0, "gu must be contiguous [M, 2F]");
+    TORCH_CHECK(!row_scale || row_scale->numel() == gu.size(0), "one scale per row");
     Tensor out = at::empty({gu.size(0), gu.size(1) / 2}, gu.options());
-    seqmix::clamped_glu(gu.data_ptr(), out.data_ptr(), is_bf(gu), gu.size(0), (int)(gu.size(1) / 2), (float)limit, (float)slope, stream());
+    seqmix::clamped_glu(gu.data_ptr(), row_scale ? f32(*row_scale) : nullptr, out.data_ptr(), is_bf(gu), gu.size(0), (int)(gu.size(1) / 2), (float)limit, (float)slope, stream());
     check_launch();
     return out;
 }

@@ -6,7 +6,8 @@
 //   on a float stream in place (gate optional), with an optional copy of the result in the sublayers' dtype.
 //   residual_norm: the joint between two sublayers of a pre-norm model, x <- x + s * y on the float stream in place and, from the new
 //   row, the next sublayer's normed input; y is a sublayer's result or the weighted sum of a routed feed-forward's expert rows, formed
-//   here (float) instead of in a launch of its own.
+//   here (float) instead of in a launch of its own.  Two norms of the same new row (two gains, one statistic) serve blocks whose
+//   sublayers run side by side; a row of a table (an embedding) and a vector may join the sum (a stretch of layers that starts again).
 #include "seq_common.cuh"
 #include "seqmix.h"
 
@@ -255,14 +256,17 @@ template <typename T, bool VEC, int NIT>
 __global__ void residual_norm_kernel(float* x, long x_stride, const T* __restrict__ y, long y_stride, const int* __restrict__ src,
                                      const float* __restrict__ weight, int top, const T* __restrict__ base,
                                      const float* __restrict__ base_weight, const float* __restrict__ scale, const float* __restrict__ w,
-                                     const float* __restrict__ bias, float eps, int center, int rows, int C, T* __restrict__ h, long h_stride) {
+                                     const float* __restrict__ bias, float eps, int center, int rows, int C, T* __restrict__ h, long h_stride,
+                                     const float* __restrict__ w2, T* __restrict__ h2, const long* __restrict__ inj_rows,
+                                     const T* __restrict__ inj_table, int inj_table_rows, const float* __restrict__ inj_vec) {
     __shared__ float part[8];
     const int row = blockIdx.x * blockDim.y + threadIdx.y, tx = threadIdx.x, TX = blockDim.x;
     const bool on = row < rows;
     const long r = on ? row : 0;
     float* xr = x + r * x_stride;
-    const T* yr = y + r * y_stride;
+    const T* yr = y ? y + r * y_stride : nullptr;
     const float bw = base_weight ? base_weight[r] : 1.f;
+    const T* ir = inj_table ? inj_table + min(max(inj_rows[r], 0L), (long)inj_table_rows - 1) * C : nullptr;
     auto row_sum = [&](float v) {               // over the threads that share the row
         v = warp_sum(v);
         if (TX > 32) {
@@ -277,15 +281,18 @@ __global__ void residual_norm_kernel(float* x, long x_stride, const T* __restric
     auto add4 = [](float4& a, float f, float4 b) { a.x = fmaf(f, b.x, a.x); a.y = fmaf(f, b.y, a.y); a.z = fmaf(f, b.z, a.z); a.w = fmaf(f, b.w, a.w); };
     auto fold4 = [&](int c, float4 s) {         // the stream's new values
         const float4 g = scale ? ld4(scale + c) : make_float4(1.f, 1.f, 1.f, 1.f), o = ld4(xr + c);
-        const float4 v = make_float4(fmaf(g.x, s.x, o.x), fmaf(g.y, s.y, o.y), fmaf(g.z, s.z, o.z), fmaf(g.w, s.w, o.w));
+        float4 v = make_float4(fmaf(g.x, s.x, o.x), fmaf(g.y, s.y, o.y), fmaf(g.z, s.z, o.z), fmaf(g.w, s.w, o.w));
+        if (ir) add4(v, 1.f, ld4(ir + c));
+        if (inj_vec) add4(v, 1.f, ld4(inj_vec + c));
         st4(xr + c, v);
         return v;
     };
     auto part4 = [&](int c) {                   // the sublayer's result
+        if (!yr) return make_float4(0.f, 0.f, 0.f, 0.f);
         if (top == 0) return ld4(yr + c);
         float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
         if (base) add4(s, bw, ld4(base + r * C + c));
-        for (int k = 0; k < top; ++k) add4(s, weight[r * top + k], ld4(y + (long)src[r * top + k] * C + c));
+        for (int k = 0; k < top; ++k) add4(s, weight ? weight[r * top + k] : 1.f, ld4(y + (long)src[r * top + k] * C + c));
         return s;
     };
     float4 kept[NIT > 0 ? NIT : 1];
@@ -294,7 +301,7 @@ __global__ void residual_norm_kernel(float* x, long x_stride, const T* __restric
         if (NIT > 0) {
             if (top == 0) {
 #pragma unroll
-                for (int i = 0; i < NIT; ++i) { const int c = (i * TX + tx) * 4; if (c < C) kept[i] = ld4(yr + c); }
+                for (int i = 0; i < NIT; ++i) { const int c = (i * TX + tx) * 4; if (c < C) kept[i] = part4(c); }
             } else {
 #pragma unroll
                 for (int i = 0; i < NIT; ++i) {
@@ -303,7 +310,7 @@ __global__ void residual_norm_kernel(float* x, long x_stride, const T* __restric
                     if (base && c < C) add4(kept[i], bw, ld4(base + r * C + c));
                 }
                 for (int k = 0; k < top; ++k) {
-                    const float f = weight[r * top + k];
+                    const float f = weight ? weight[r * top + k] : 1.f;
                     const T* er = y + (long)src[r * top + k] * C;
 #pragma unroll
                     for (int i = 0; i < NIT; ++i) { const int c = (i * TX + tx) * 4; if (c < C) add4(kept[i], f, ld4(er + c)); }
@@ -319,12 +326,15 @@ __global__ void residual_norm_kernel(float* x, long x_stride, const T* __restric
         } else {
             for (int c = tx; c < C; c += TX) {
                 float s;
-                if (top == 0) s = ldf(yr + c);
+                if (!yr) s = 0.f;
+                else if (top == 0) s = ldf(yr + c);
                 else {
                     s = base ? bw * ldf(base + r * C + c) : 0.f;
-                    for (int k = 0; k < top; ++k) s = fmaf(weight[r * top + k], ldf(y + (long)src[r * top + k] * C + c), s);
+                    for (int k = 0; k < top; ++k) s = fmaf(weight ? weight[r * top + k] : 1.f, ldf(y + (long)src[r * top + k] * C + c), s);
                 }
-                const float v = fmaf(scale ? scale[c] : 1.f, s, xr[c]);
+                float v = fmaf(scale ? scale[c] : 1.f, s, xr[c]);
+                if (ir) v += ldf(ir + c);
+                if (inj_vec) v += inj_vec[c];
                 xr[c] = v;
                 sx += v;
             }
@@ -355,6 +365,10 @@ __global__ void residual_norm_kernel(float* x, long x_stride, const T* __restric
         const float4 g = ld4(w + c), u = bias ? ld4(bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
         st4(hr + c, make_float4((v.x - mean) * inv * g.x + u.x, (v.y - mean) * inv * g.y + u.y, (v.z - mean) * inv * g.z + u.z,
                                 (v.w - mean) * inv * g.w + u.w));
+        if (w2) {
+            const float4 k = ld4(w2 + c);
+            st4(h2 + r * C + c, make_float4((v.x - mean) * inv * k.x, (v.y - mean) * inv * k.y, (v.z - mean) * inv * k.z, (v.w - mean) * inv * k.w));
+        }
     };
     if (NIT > 0) {
 #pragma unroll
@@ -362,24 +376,30 @@ __global__ void residual_norm_kernel(float* x, long x_stride, const T* __restric
     } else if (VEC) {
         for (int c = tx * 4; c < C; c += TX * 4) put4(c, ld4(xr + c));
     } else {
-        for (int c = tx; c < C; c += TX) stf(hr + c, (xr[c] - mean) * inv * w[c] + (bias ? bias[c] : 0.f));
+        for (int c = tx; c < C; c += TX) {
+            const float v = (xr[c] - mean) * inv;
+            stf(hr + c, v * w[c] + (bias ? bias[c] : 0.f));
+            if (w2) stf(h2 + r * C + c, v * w2[c]);
+        }
     }
 }
 
 void residual_norm(float* x, long x_stride, const void* y, long y_stride, int bf, const int* src, const float* weight, int top, const void* base,
                    const float* base_weight, const float* scale, const float* w, const float* bias, float eps, int center, int rows, int C,
-                   void* h, long h_stride, cudaStream_t s) {
+                   void* h, long h_stride, const float* w2, void* h2, const long* inj_rows, const void* inj_table, int inj_table_rows,
+                   const float* inj_vec, cudaStream_t s) {
     if (rows == 0) return;
     const bool few = C >= 1024 || (rows < 148 * 8 && C >= 512);
     dim3 block(few ? 256 : 32, few ? 1 : 8), grid(few ? rows : (rows + 7) / 8);
     const size_t e = bf ? 2 : 4;
     auto al = [](const void* p, size_t b) { return p == nullptr || (uintptr_t)p % b == 0; };
     const bool vec = C % 4 == 0 && x_stride % 4 == 0 && y_stride % 4 == 0 && (!w || h_stride % 4 == 0) && al(x, 16) && al(w, 16) && al(bias, 16) &&
-                     al(scale, 16) && al(y, 4 * e) && al(base, 4 * e) && al(h, 4 * e);
+                     al(scale, 16) && al(y, 4 * e) && al(base, 4 * e) && al(h, 4 * e) && al(w2, 16) && al(h2, 4 * e) && al(inj_table, 4 * e) && al(inj_vec, 16);
     const int per = vec ? (C / 4 + (int)block.x - 1) / (int)block.x : 0;
 #define SEQMIX_RN(T, V, N)                                                                                                           \
     residual_norm_kernel<T, V, N><<<grid, block, 0, s>>>(x, x_stride, (const T*)y, y_stride, src, weight, top, (const T*)base, base_weight,  \
-                                                         scale, w, bias, eps, center, rows, C, (T*)h, h_stride)
+                                                         scale, w, bias, eps, center, rows, C, (T*)h, h_stride, w2, (T*)h2, inj_rows,             \
+                                                         (const T*)inj_table, inj_table_rows, inj_vec)
 #define SEQMIX_RN_T(T)                                                                                                               \
     do {                                                                                                                             \
         if (!vec) SEQMIX_RN(T, false, 0);                                                                                            \

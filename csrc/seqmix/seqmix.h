@@ -10,10 +10,13 @@ void rms_norm(const void* x, int in_bf16, long x_stride, int rows, int C, const 
               long gate_stride, void* out, int out_bf16, long out_stride, float* res, long res_stride, int center, const float* bias,
               cudaStream_t s);
 // x (float, in place) += scale * y, then (w given) h <- norm(x) * w + bias; y [rows, C], or with top > 0 the expert rows whose weighted
-// sums (weight, src [rows, top]; base times base_weight added) take its place.  scale, bias, base, base_weight, w may be null.
+// sums (weight, src [rows, top], weight null: plain sums; base times base_weight added) take its place.  scale, bias, base, base_weight,
+// w and y (null: nothing is added) may be null.  w2: a second gain for the same statistics, its result in h2.  inj_table ([*, C] of h's
+// dtype, row inj_rows[row]) and inj_vec [C] are added to x as well, after the scaled sum.
 void residual_norm(float* x, long x_stride, const void* y, long y_stride, int bf, const int* src, const float* weight, int top, const void* base,
                    const float* base_weight, const float* scale, const float* w, const float* bias, float eps, int center, int rows, int C,
-                   void* h, long h_stride, cudaStream_t s);
+                   void* h, long h_stride, const float* w2, void* h2, const long* inj_rows, const void* inj_table, int inj_table_rows,
+                   const float* inj_vec, cudaStream_t s);
 // x (float, in place) <- norm(alpha * x + sigmoid(gate) * y) * w; gate may be null; lp (of y's dtype, may be null) gets a copy
 void postnorm_gated(float* x, long x_stride, const void* y, long y_stride, const void* gate, long gate_stride, int bf, const float* w,
                     float alpha, float eps, int rows, int C, void* lp, long lp_stride, cudaStream_t s);
@@ -75,14 +78,16 @@ void xielu(const void* x, void* out, int bf, long n, float ap, float an, cudaStr
 void relu_sq(const void* x, void* out, int bf, long n, cudaStream_t s);
 void gelu_erf(const void* x, void* out, int bf, long n, cudaStream_t s);
 void silu_mul(const void* gu, void* out, int bf, long rows, int F, cudaStream_t s);
-void clamped_glu(const void* gu, void* out, int bf, long rows, int F, float limit, float slope, cudaStream_t s);
+// row_scale (one float per row, or null) multiplies the row before the activation
+void clamped_glu(const void* gu, const float* row_scale, void* out, int bf, long rows, int F, float limit, float slope, cudaStream_t s);
 void sigmoid_gate_mul(void* x, int bf, const void* gate, int gate_bf, long gate_stride, long rows, int C, int rep, cudaStream_t s);
 void rotary_qkv_f32(const void* p, int bf, long p_sb, long p_st, int B, int S, int C, int hq, int hk, int D, int dims,
                     const float* inv_freq, const int* pos0, float q_scale, float k_scale, float* out, cudaStream_t s);
 // act 0: none, 1: gelu_erf, 2: silu(gate rows . x) * (up rows . x) with the gate rows stacked over the up rows (O/2 outputs),
-// 3: the square of relu
-void indexed_gemv(const void* w, const int* sel, const void* x, int bf, long x_stride, int M, int E, int O, int I, int act, void* out,
-                  cudaStream_t s);
+// 3: the square of relu, 4: like 2 with the clamped gate of clamped_glu (limit, slope); x_scale (one float per row, or null) multiplies x
+void indexed_gemv(const void* w, const int* sel, const void* x, int bf, long x_stride, const float* x_scale, int M, int E, int O, int I, int act,
+                  float limit, float slope, void* out, cudaStream_t s);
+// weight null: plain sums
 void moe_combine(const void* rows, const int* src, const float* weight, const void* base, const float* base_weight, int bf, int N, int top,
                  int C, void* out, cudaStream_t s);
 // false: more experts than the kernel takes (256)
@@ -99,29 +104,49 @@ void embed_bigram(const long* tokens, const void* table, int bf, float scale, co
 void group_rms_norm_gated(const void* x, int in_bf16, long x_stride, const void* gate, int gate_bf16, long gate_stride, const float* w,
                           int wn, int rows, int C, int groups, float eps, int gate_first, void* out, long out_stride, float out_scale,
                           int sigmoid_gate, cudaStream_t s);
-// Grouped-query sliding-window attention (window_attention.cu); false: sizes do not fit (value size above 512).
-// window_qk_prepare: norm_all 0: an RMS norm per head (qw, kw hold D numbers), 1: one over all heads (H*D and G*D numbers); inv_freq
-// (dims/2 numbers, or null): rotation of the first dims coordinates; k null: only the queries are prepared.
-// score_bias (one float per query head, or null): sigmoid(score + bias) weights, not normalised, instead of a softmax.
-void window_qk_prepare(void* q, long q_sb, long q_st, void* k, long k_sb, long k_st, const void* v, long v_sb, long v_st, int bf,
-                       const float* qw, const float* kw, int norm_all, float eps, const float* inv_freq, int dims, const int* pos0,
-                       const int* lens, const int* slots, void* kcache, void* vcache, int ring, int B, int S, int H, int G, int D, int V,
-                       cudaStream_t s);
+// Grouped-query attention over a window, a chunk or the whole sequence (window_attention.cu); false: sizes do not fit (value size above 512).
+struct WindowRule {
+    int window;                  // position i sees j with i - j < window ...
+    int chunk;                   // ... and, when > 0, i / chunk == j / chunk
+    float scale, softcap;        // score = q.k * scale, capped when softcap > 0
+    const float* score_bias;     // one per query head, or null: sigmoid(score + bias) weights, not normalised, instead of a softmax
+    const float* sink;           // one per query head and map, or null: exp(sink) joins the softmax's denominator
+    int maps;                    // 1, or 2: a head's result is unit(a1 - lam[0] * a2) * post, unit(o) = o / sqrt(mean(o^2) + eps)
+    const float* lam;
+    float eps, post;
+};
+// window_qk_prepare: H query heads, GK key heads (maps counted), G value heads; norm_all 0: an RMS norm per head (qw, kw hold D numbers),
+// 1: one over all heads (H*D and GK*D numbers); unit: a norm without weights AFTER the rotation; inv_freq (dims/2 numbers, or null):
+// rotation of the first dims coordinates, cos and sin times amp; kout: where the prepared keys go (k itself, or another tensor when
+// v aliases k); k null: only the queries are prepared.
+void window_qk_prepare(void* q, long q_sb, long q_st, void* k, long k_sb, long k_st, void* kout, long ko_sb, long ko_st, const void* v,
+                       long v_sb, long v_st, int bf, const float* qw, const float* kw, int norm_all, int unit, float eps,
+                       const float* inv_freq, int dims, float amp, const int* pos0, const int* lens, const int* slots, void* kcache,
+                       void* vcache, int ring, int B, int S, int H, int GK, int G, int D, int V, cudaStream_t s);
+// H heads of the rule's maps (q [B,S,H*maps,D], k [B,S,G*maps,D], v [B,S,G,V]).  maps_room: float [B*S, H, 2, V], needed with two maps
+// unless window_prompt_fused says that the tensor-core kernel takes the call.
+bool window_prompt_fused(const void* q, long q_sb, long q_st, const void* k, long k_sb, long k_st, const void* v, long v_sb, long v_st, int bf,
+                         int D, int V, int maps, const void* out, long out_stride);
 bool window_attention_prompt(const void* q, long q_sb, long q_st, const void* k, long k_sb, long k_st, const void* v, long v_sb, long v_st,
                              const void* gate, long g_sb, long g_st, int bf, const int* lens, int B, int S, int H, int G, int D, int V,
-                             int window, float scale, float softcap, const float* score_bias, void* out, long out_stride, float out_scale,
-                             cudaStream_t s);
+                             const WindowRule& rule, float* maps_room, void* out, long out_stride, float out_scale, cudaStream_t s);
 bool window_prompt_mma_fits(const void* q, long q_sb, long q_st, const void* k, long k_sb, long k_st, const void* v, long v_sb, long v_st,
-                            int D, int V, const void* out, long out_stride);
+                            int D, int V, int maps, const void* out, long out_stride);
 void window_prompt_mma(const void* q, long q_sb, long q_st, const void* k, long k_sb, long k_st, const void* v, long v_sb, long v_st,
-                       const void* gate, long g_sb, long g_st, const int* lens, int B, int S, int H, int G, int D, int V, int window,
-                       float scale, float softcap, const float* score_bias, void* out, long out_stride, float out_scale, cudaStream_t s);
-// part_m / part_l float [B, H, splits], part_acc float [B, H, splits, V] with splits = window_token_splits(...)
-int window_token_splits(int ring, int B, int H, int G);
+                       const void* gate, long g_sb, long g_st, const int* lens, int B, int S, int H, int G, int D, int V,
+                       const WindowRule& rule, void* out, long out_stride, float out_scale, cudaStream_t s);
+// part_m / part_l float [B, H*maps, splits], part_acc float [B, H*maps, splits, V] with splits = window_token_splits(...)
+int window_token_splits(int ring, int bf, int B, int H, int G, int D, int V, const WindowRule& rule);
 bool window_attention_token(const void* q, long q_sb, const void* kcache, const void* vcache, const void* gate, long g_sb, int bf,
-                            const int* slots, const int* pos0, const int* lens, int ring, int B, int H, int G, int D, int V, int window,
-                            float scale, float softcap, const float* score_bias, int splits, float* part_m, float* part_l, float* part_acc,
-                            void* out, long out_stride, float out_scale, cudaStream_t s);
+                            const int* slots, const int* pos0, const int* lens, int ring, int B, int H, int G, int D, int V,
+                            const WindowRule& rule, int splits, float* part_m, float* part_l, float* part_acc, void* out, long out_stride,
+                            float out_scale, cudaStream_t s);
+// The tensor-core form of its first kernel (window_decode_mma.cu; bfloat16, softmax without a cap).
+bool window_decode_mma_fits(int D, int V, int maps);
+int window_decode_mma_splits(int B, int H, int G, int D, int V, int maps, int rows);
+void window_decode_mma(const void* q, long q_sb, const void* kcache, const void* vcache, const int* slots, const int* pos0, const int* lens,
+                       int ring, int B, int H, int G, int D, int V, const WindowRule& rule, int splits, float* part_m, float* part_l,
+                       float* part_acc, cudaStream_t s);
 // Matrix-state recurrences with one decay per head and token (matrix_recurrence.cu); false: the state has too many rows.
 bool gated_delta_scan(const void* q, const void* k, long qk_sb, long qk_st, const void* v, long v_sb, long v_st, int bf, const float* braw,
                       const float* araw, long ba_sb, long ba_st, const float* a_log, const float* dt_bias, float* state, const int* slots,
