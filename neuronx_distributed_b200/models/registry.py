@@ -66,6 +66,12 @@ def _load_kulisun(model_dir, dtype, device, max_seq_len, batch_size, **kw):
     return KulisunForInference.from_pretrained(model_dir, dtype=dtype, device=device, max_seq_len=max_seq_len, batch_size=batch_size, **kw)
 
 
+def _load_kekelix(model_dir, dtype, device, max_seq_len, batch_size, **kw):
+    from .kekelix import KekelixForInference
+
+    return KekelixForInference.from_pretrained(model_dir, dtype=dtype, device=device, max_seq_len=max_seq_len, batch_size=batch_size, **kw)
+
+
 def _load_hf_decoder(model_dir, dtype, device, max_seq_len, batch_size, **kw):
     """Llama / Mistral / Mixtral / DBRX checkpoints (model-parallel state must be initialised by the caller)."""
     from . import hf_compat
@@ -85,5 +91,6 @@ register_family("pinirax", _load_pinirax)
 register_family("pulenex", _load_pulenex)
 register_family("noresun", _load_noresun)
 register_family("kulisun", _load_kulisun)
+register_family("kekelix", _load_kekelix)
 for _name in ("llama", "mistral", "qwen2", "mixtral", "dbrx"):
     register_family(_name, _load_hf_decoder)

@@ -13,6 +13,11 @@ worth the sum of its two largest scores).  ``renormalise``: the chosen scores ar
 expert has the gated form (``shared_up [2 shared_ff, width]``: gate rows over up rows).  ``shared_gate``: the shared expert's output is
 multiplied by ``sigmoid(w . h)``, one number per token; that row rides on the router's product as its last one.
 
+``glu = (limit, slope)``: the gated experts' activation is ``g sigmoid(slope g) (u + 1)`` with ``g = min(gate, limit)`` and ``u`` clamped to
+``[-limit, limit]`` instead of ``silu(gate) * up``.  ``weigh_input``: a chosen expert's weight multiplies what the expert READS,
+``sum_e expert_e(s_e h)``; the gate and up products are linear, so the weight enters as a number per row of the activation's input and the
+rows are summed without weights.
+
 Two more options of the router.  ``choice_bias``: a float vector added to the scores for the CHOICE only (the weights stay the plain
 scores).  ``identity_experts``: the router's last outputs name experts without tensors whose output is the input itself; their
 weights are summed per token and enter the combine as a weighted copy of the input.
@@ -41,8 +46,12 @@ class RoutedFFN(nn.Module):
     def __init__(self, width: int, ff: int, experts: int, top: int, weight_scale: float = 1.0, shared_ff: int = 0,
                  router_act: str = "sigmoid", gated: bool = False, identity_experts: int = 0, choice_bias: bool = False,
                  dtype: torch.dtype = torch.bfloat16, device=None, router_bias: bool = False, expert_act: str = "gelu",
-                 groups=None, renormalise: bool = False, shared_gated: bool = False, shared_gate: bool = False):
+                 groups=None, renormalise: bool = False, shared_gated: bool = False, shared_gate: bool = False,
+                 glu=None, weigh_input: bool = False):
         super().__init__()
+        assert glu is None or gated, "a clamped gate belongs to gated experts"
+        assert not weigh_input or (glu is not None and not identity_experts), "weights on the experts' input: clamped gated experts only"
+        self.glu, self.weigh_input = None if glu is None else (float(glu[0]), float(glu[1])), weigh_input
         assert not shared_gate or (shared_ff and not identity_experts), "a gate needs a shared expert (and identity experts take its place)"
         assert expert_act in ("gelu", "relu_sq"), expert_act
         assert router_act != "softmax_top" or not (identity_experts or choice_bias), "softmax over the chosen logits: plain experts only"
@@ -93,8 +102,11 @@ class RoutedFFN(nn.Module):
                                           self.weight_scale, self.groups, self.renormalise, self.shared_gate)
         return w, idx, (ident if self.identity_experts or self.shared_gate else None)
 
-    def _act(self, y: torch.Tensor) -> torch.Tensor:
-        """The experts' activation on the up-projection's output: ``[M, ff]`` (plain) or ``[M, 2 ff]`` → ``[M, ff]`` (gated)."""
+    def _act(self, y: torch.Tensor, row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The experts' activation on the up-projection's output: ``[M, ff]`` (plain) or ``[M, 2 ff]`` → ``[M, ff]`` (gated).
+        ``row_scale [M]``: the weights of experts that weigh their input."""
+        if self.glu is not None:
+            return seqmix.clamped_glu(y, *self.glu, row_scale)
         if self.gated:
             return seqmix.silu_mul(y)
         return seqmix.relu_sq(y) if self.expert_act == "relu_sq" else seqmix.gelu_erf(y)
@@ -110,7 +122,7 @@ class RoutedFFN(nn.Module):
         e = _ext.ext()
         return e if e is not None and hasattr(e, "grouped_gemm") else None
 
-    def _experts_grouped(self, h: torch.Tensor, idx: torch.Tensor):
+    def _experts_grouped(self, h: torch.Tensor, idx: torch.Tensor, in_w: Optional[torch.Tensor] = None):
         """All chosen experts in two grouped GEMMs over the blockwise layout → (rows ``[blocks * 128, width]``, ``src [N, top]``
         naming the row that holds each (token, choice)).  Padding slots compute on token 0 and are never referenced."""
         from ...ops import _ext
@@ -127,10 +139,11 @@ class RoutedFFN(nn.Module):
         tp = tp2id[: b2e.numel() * bs].long()
         x = h[tp.clamp(min=0)]
         _ext.count_launch(2)
-        eo = e.grouped_gemm(self._act(e.grouped_gemm(x, self.up, b2e, bs, True)), self.down, b2e, bs, True)
         N, top = idx.shape                                                         # no host synchronisation: padding slots write
         tok, exp = tp.clamp(min=0), group.repeat_interleave(bs)                    # to a spare entry past the end
         choice = (idx[tok] == exp[:, None]).to(torch.int32).argmax(1)
+        scale = None if in_w is None else in_w[tok, choice]
+        eo = e.grouped_gemm(self._act(e.grouped_gemm(x, self.up, b2e, bs, True), scale), self.down, b2e, bs, True)
         flat = torch.empty(N * top + 1, dtype=torch.int32, device=h.device)
         flat[torch.where(tp >= 0, tok * top + choice, N * top)] = torch.arange(tp.numel(), dtype=torch.int32, device=h.device)
         src = flat[: N * top].view(N, top)
@@ -148,14 +161,17 @@ class RoutedFFN(nn.Module):
         does its work, ``seqmix.residual_norm_``) adds up."""
         N = h.shape[0]
         w, idx, ident_w = self.route(h)                            # identity choices: weight 0, their scores summed in ident_w
+        in_w = w if self.weigh_input else None
         M = N * self.top
         if M <= self.small_batch_rows:
             sel = idx.reshape(-1).to(torch.int32)                  # the streaming kernels skip rows that name no matrix
-            mid = seqmix.indexed_gemv(self.up, sel, h.repeat_interleave(self.top, 0), "silu_glu" if self.gated else self.expert_act)
+            act = "clamped_glu" if self.glu is not None else ("silu_glu" if self.gated else self.expert_act)
+            mid = seqmix.indexed_gemv(self.up, sel, h.repeat_interleave(self.top, 0) if self.top > 1 else h, act,
+                                      None if in_w is None else in_w.reshape(-1), *(self.glu or ()))
             eo = seqmix.indexed_gemv(self.down, sel, mid, None)
             src = torch.arange(M, device=h.device, dtype=torch.int32).view(N, self.top)
         elif self._grouped_kernels(h) is not None:
-            eo, src = self._experts_grouped(h, idx)
+            eo, src = self._experts_grouped(h, idx, in_w)
         else:
             flat = idx.reshape(-1)
             order = torch.argsort(flat, stable=True)
@@ -163,10 +179,12 @@ class RoutedFFN(nn.Module):
             xs = h[order // self.top]
             eo = torch.zeros(M, self.width, dtype=h.dtype, device=h.device) if self.identity_experts else \
                 torch.empty(M, self.width, dtype=h.dtype, device=h.device)
+            ws = None if in_w is None else in_w.reshape(-1)[order]
             off = 0
             for e, c in enumerate(counts):
                 if c:
-                    eo[off:off + c] = F.linear(self._act(F.linear(xs[off:off + c], self.up[e])), self.down[e])
+                    mid = self._act(F.linear(xs[off:off + c], self.up[e]), None if ws is None else ws[off:off + c])
+                    eo[off:off + c] = F.linear(mid, self.down[e])
                     off += c
             src = torch.empty(M, dtype=torch.int32, device=h.device)
             src[order] = torch.arange(M, device=h.device, dtype=torch.int32)
@@ -179,4 +197,4 @@ class RoutedFFN(nn.Module):
         if self.shared_ff:
             mid = F.linear(h, self.shared_up)
             base = F.linear(seqmix.silu_mul(mid) if self.shared_gated else seqmix.gelu_erf(mid), self.shared_down)
-        return eo, (src, w.contiguous(), base, ident_w if self.shared_gate else None)
+        return eo, (src, None if self.weigh_input else w.contiguous(), base, ident_w if self.shared_gate else None)

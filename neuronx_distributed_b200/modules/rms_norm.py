@@ -86,8 +86,9 @@ class ScalarRMSNorm(nn.Module):
 class OffsetRMSNorm(nn.Module):
     """RMS norm whose checkpoint stores the gain's offset from one: ``x / sqrt(mean(x^2) + eps) * (1 + w)``.  The parameter here
     is the gain itself, ``1 + w`` formed once in float (``set_offset``).  ``forward`` gives the sublayer's input in ``out_dtype``;
-    ``add_to(res, y)`` is the closing norm of a sandwich block, ``res += norm(y)`` with ``res`` a float stream (one kernel each,
-    ``csrc/seqmix/norms.cu``)."""
+    ``add_to(res, y)`` is the closing norm of a sandwich block, ``res += norm(y)`` with ``res`` a float stream; ``after_sum`` is the norm
+    joined with the residual sum before it, ``second`` another norm of the same new rows (``ops.seqmix.residual_norm_``; one kernel
+    each, ``csrc/seqmix/norms.cu``)."""
 
     def __init__(self, width: int, eps: float = 1e-6, device=None):
         super().__init__()
@@ -109,6 +110,13 @@ class OffsetRMSNorm(nn.Module):
 
         seqmix.add_rms_norm_(res.view(-1, res.shape[-1]), y.reshape(-1, y.shape[-1]), self.weight, self.eps)
         return res
+
+    def after_sum(self, x: torch.Tensor, y: Optional[torch.Tensor], experts=None, second: Optional["OffsetRMSNorm"] = None, inject=None,
+                  out_dtype: Optional[torch.dtype] = None):
+        from ..ops import seqmix
+
+        return seqmix.residual_norm_(x, y, None, self.weight, None, self.eps, False, experts, None if second is None else second.weight, inject,
+                                     out_dtype)
 
 
 class GainOnlyLayerNorm(nn.Module):

@@ -1,7 +1,7 @@
 """Sequence-mixer ops: short causal convolutions with carried history, scalar / vector RMS and layer norms (optionally accumulated
 into a float residual stream, closing a block whose norm follows a gated residual sum, or joined with the residual sum before them), token embeddings with sinusoids or a hashed
-pair table, latent / grouped-query / head-mixing attention over ring caches (sliding window or the whole sequence; softmax, with or
-without a sink, or independent sigmoid weights),
+pair table, latent / grouped-query / head-mixing attention over ring caches (sliding window, aligned chunks or the whole sequence; softmax,
+with or without a sink, the difference of two softmax maps, or independent sigmoid weights),
 gated linear recurrences (per-key-channel decay; real-gated LRU; minGRU), matrix-state recurrences, xIELU / erf-GELU / squared relu
 and the small-batch pieces of a routed feed-forward.
 
@@ -41,7 +41,7 @@ GROUPS = {
     "linrec": (["linear_recurrence.cu", "gla_chunked.cu", "bind_linrec.cpp"], ["gla_scan", "rglru_scan", "retention_scan", "mingru_scan"]),
     "headmix": (["headmix_attention.cu", "headmix_decode.cu", "headmix_prefill.cu", "bind_headmix.cpp"],
                 ["headmix_qk_prepare", "headmix_attention_prompt", "headmix_attention_token"]),
-    "window": (["window_attention.cu", "window_prefill.cu", "bind_window.cpp"], ["window_qk_prepare", "window_attention_prompt", "window_attention_token"]),
+    "window": (["window_attention.cu", "window_decode_mma.cu", "window_prefill.cu", "bind_window.cpp"], ["window_qk_prepare", "window_attention_prompt", "window_attention_token"]),
     "matrec": (["matrix_recurrence.cu", "bind_matrec.cpp"], ["gated_delta_scan", "ssd_scan"]),
 }
 _GROUP_OF = {fn: g for g, (_, fns) in GROUPS.items() for fn in fns}
@@ -196,25 +196,41 @@ def postnorm_gated_(x: torch.Tensor, y: torch.Tensor, gate: Optional[torch.Tenso
     return x
 
 
-def residual_norm_(x: torch.Tensor, y: torch.Tensor, scale: Optional[torch.Tensor], w: Optional[torch.Tensor], bias: Optional[torch.Tensor],
-                   eps: float, center: bool = False, experts=None) -> Optional[torch.Tensor]:
+def residual_norm_(x: torch.Tensor, y: Optional[torch.Tensor], scale: Optional[torch.Tensor], w: Optional[torch.Tensor], bias: Optional[torch.Tensor],
+                   eps: float, center: bool = False, experts=None, w2: Optional[torch.Tensor] = None, inject=None,
+                   out_dtype: Optional[torch.dtype] = None):
     """The joint between two sublayers of a pre-norm model, one launch: the float stream ``x [rows, C]`` gets ``x += scale * y`` in place
-    (``scale [C]`` float or None) and the new rows' norm ``norm(x) * w + bias`` comes back in ``y``'s dtype (``center``: a layer norm,
-    otherwise an RMS norm; ``w`` None: no norm, returns None).  ``experts = (src, weight, base, base_weight)``: ``y`` holds a routed
-    feed-forward's expert rows ``[M, C]`` and ``sum_k weight[n,k] * y[src[n,k]] (+ base_weight[n] * base[n])``, summed in float, takes
-    its place."""
+    (``scale [C]`` float or None; ``y`` None: nothing) and the new rows' norm ``norm(x) * w + bias`` comes back in ``y``'s dtype
+    (``out_dtype`` without a ``y``; ``center``: a layer norm, otherwise an RMS norm; ``w`` None: no norm, returns None).  ``experts =
+    (src, weight, base, base_weight)``: ``y`` holds a routed feed-forward's expert rows ``[M, C]`` and ``sum_k weight[n,k] * y[src[n,k]]
+    (+ base_weight[n] * base[n])``, summed in float, takes its place (``weight`` None: ones).  ``inject = (rows, table, vec)``: ``table[rows[n]]``
+    (int64 ``rows``, ``table`` of the result's dtype; both None: nothing) and ``vec [C]`` (float or None) are added to the stream as well.
+    ``w2``: a second gain for the same statistic; the result is then the pair of both norms."""
     src, weight, base, base_weight = experts if experts is not None else (None, None, None, None)
+    irows, itable, ivec = inject if inject is not None else (None, None, None)
+    dtype = y.dtype if y is not None else out_dtype or (itable.dtype if itable is not None else x.dtype)
     if _cuda(x):
         _ext.count_launch()
-        h = ext().residual_norm_(x, y, scale, w, bias, float(eps), center, None if src is None else _i32(src), weight, base, base_weight)
-        return h if w is not None else None
-    v = y.float()
-    if src is not None:
-        v = (v[src.long()] * weight[..., None]).sum(1)
-        if base is not None:
-            v = v + (base.float() if base_weight is None else base.float() * base_weight[:, None])
-    x += v if scale is None else scale * v
-    return None if w is None else rms_norm(x, w, eps, None, y.dtype, center, bias)
+        like = y if y is not None else torch.empty(0, dtype=dtype, device=x.device)
+        h, h2 = ext().residual_norm_(x, y, scale, w, bias, float(eps), center, None if src is None else _i32(src), weight, base, base_weight, w2,
+                                     irows, itable, ivec, like)
+        return None if w is None else (h if w2 is None else (h, h2))
+    if y is not None:
+        v = y.float()
+        if src is not None:
+            v = v[src.long()]
+            v = (v if weight is None else v * weight[..., None]).sum(1)
+            if base is not None:
+                v = v + (base.float() if base_weight is None else base.float() * base_weight[:, None])
+        x += v if scale is None else scale * v
+    if irows is not None:
+        x += itable[irows.reshape(-1).clamp(0, itable.shape[0] - 1)].float()
+    if ivec is not None:
+        x += ivec
+    if w is None:
+        return None
+    h = rms_norm(x, w, eps, None, dtype, center, bias)
+    return h if w2 is None else (h, rms_norm(x, w2, eps, None, dtype, center))
 
 
 # ---------------------------------------------------------------------------------------------------------------- latent attention
@@ -543,19 +559,23 @@ def relu_sq(x: torch.Tensor) -> torch.Tensor:
     return torch.relu(x.float()).pow(2).to(x.dtype)
 
 
-GEMV_ACTS = {None: 0, "none": 0, "gelu": 1, "silu_glu": 2, "relu_sq": 3}
+GEMV_ACTS = {None: 0, "none": 0, "gelu": 1, "silu_glu": 2, "relu_sq": 3, "clamped_glu": 4}
 
 
-def indexed_gemv(w: torch.Tensor, sel: torch.Tensor, x: torch.Tensor, act) -> torch.Tensor:
+def indexed_gemv(w: torch.Tensor, sel: torch.Tensor, x: torch.Tensor, act, x_scale: Optional[torch.Tensor] = None, limit: float = 0.0,
+                 slope: float = 1.0) -> torch.Tensor:
     """``w [E,O,I]``, ``sel [M]``, ``x [M,I]`` → ``act(w[sel[m]] @ x[m])`` (float accumulation).  ``act``: ``None``, ``"gelu"`` (erf
-    form; ``True`` means the same), ``"relu_sq"`` (the square of relu) or ``"silu_glu"``: the matrix stacks gate rows over up rows and the result is
-    ``silu(gate) * up``, ``[M, O/2]``.  Rows whose ``sel`` names no matrix (``< 0`` or ``>= E``) give zeros."""
+    form; ``True`` means the same), ``"relu_sq"`` (the square of relu), ``"silu_glu"``: the matrix stacks gate rows over up rows and the result is
+    ``silu(gate) * up``, ``[M, O/2]``, or ``"clamped_glu"``: the same with :func:`clamped_glu` of ``limit`` and ``slope``.  ``x_scale [M]``
+    (float): ``act(w[sel[m]] @ (x_scale[m] x[m]))``.  Rows whose ``sel`` names no matrix (``< 0`` or ``>= E``) give zeros."""
     kind = GEMV_ACTS["gelu" if act is True else (None if act is False else act)]
     if _cuda(x):
         _ext.count_launch()
-        return ext().indexed_gemv(w, _i32(sel), x, kind)
+        return ext().indexed_gemv(w, _i32(sel), x, kind, x_scale, float(limit), float(slope))
     ok = (sel >= 0) & (sel < w.shape[0])
     y = torch.einsum("moi,mi->mo", w[sel.long().clamp(0, w.shape[0] - 1)].float(), x.float())
+    if x_scale is not None:
+        y = y * x_scale.reshape(-1, 1)
     if kind == 1:
         y = F.gelu(y)
     elif kind == 2:
@@ -563,6 +583,8 @@ def indexed_gemv(w: torch.Tensor, sel: torch.Tensor, x: torch.Tensor, act) -> to
         y = F.silu(y[:, :half]) * y[:, half:]
     elif kind == 3:
         y = torch.relu(y).pow(2)
+    elif kind == 4:
+        y = clamped_glu(y, limit, slope)
     return torch.where(ok[:, None], y, torch.zeros_like(y)).to(x.dtype)
 
 
@@ -575,14 +597,15 @@ def silu_mul(gu: torch.Tensor) -> torch.Tensor:
     return (F.silu(gu[:, :half].float()) * gu[:, half:].float()).to(gu.dtype)
 
 
-def moe_combine(rows: torch.Tensor, src: torch.Tensor, weight: torch.Tensor, base: Optional[torch.Tensor],
+def moe_combine(rows: torch.Tensor, src: torch.Tensor, weight: Optional[torch.Tensor], base: Optional[torch.Tensor],
                 base_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out[n] = base_weight[n] * base[n] + sum_k weight[n,k] * rows[src[n,k]]`` summed in float; ``rows [M,C]``, ``src, weight
-    [N,top]``, ``base [N,C]`` (optional; ``base_weight [N]`` float, one when absent)."""
+    [N,top]`` (``weight`` None: ones), ``base [N,C]`` (optional; ``base_weight [N]`` float, one when absent)."""
     if _cuda(rows):
         _ext.count_launch()
         return ext().moe_combine(rows, _i32(src), weight, base, base_weight)
-    y = (rows.float()[src.long()] * weight[..., None]).sum(1)
+    y = rows.float()[src.long()]
+    y = (y if weight is None else y * weight[..., None]).sum(1)
     if base is not None:
         y = y + (base.float() if base_weight is None else base.float() * base_weight[:, None])
     return y.to(rows.dtype)
@@ -664,22 +687,26 @@ def group_rms_norm_gated(x: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, g
     return out
 
 
-# ------------------------------------------------------------------------------------- grouped-query sliding-window attention
+# --------------------------------------------------------------- grouped-query attention (window, aligned chunk or whole sequence)
 def window_qk_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], qw: Optional[torch.Tensor],
                       kw: Optional[torch.Tensor], eps: float, pos0: torch.Tensor, lens: torch.Tensor, slots: torch.Tensor,
                       kcache: Optional[torch.Tensor], vcache: Optional[torch.Tensor], norm_all: bool = False,
-                      inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0) -> None:
-    """``q [B,S,H,D]``, ``k [B,S,G,D]``, ``v [B,S,G,V]`` (views; last dim contiguous), all IN PLACE.  Norm: every head's query and key
+                      inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0, amp: float = 1.0, unit: bool = False,
+                      kout: Optional[torch.Tensor] = None) -> None:
+    """``q [B,S,H,D]``, ``k [B,S,GK,D]``, ``v [B,S,G,V]`` (views; last dim contiguous; ``GK`` is G or, with two score maps, 2 G), IN PLACE.
+    Norm: every head's query and key
     is divided by its root mean square and multiplied by ``qw`` / ``kw`` (``[D]`` float; ``None``: left as they are); with
     ``norm_all`` the root mean square is taken over ALL heads of the token's queries (keys) at once and the weights hold ``H*D``
-    (``G*D``) numbers.  Rotation (``inv_freq [rot_dims/2]`` given): afterwards the first ``rot_dims`` coordinates of every query and
-    key head are rotated at position ``pos0[b] + t``, coordinate ``i`` paired with ``i + rot_dims/2``, angles in float.  The last
-    ``ring`` real tokens of each row go to ``kcache [slots, ring, G, D]`` / ``vcache [slots, ring, G, V]`` at row
+    (``GK*D``) numbers.  Rotation (``inv_freq [rot_dims/2]`` given): afterwards the first ``rot_dims`` coordinates of every query and
+    key head are rotated at position ``pos0[b] + t``, coordinate ``i`` paired with ``i + rot_dims/2``, angles in float, cos and sin times
+    ``amp``.  ``unit``: no weights, and the norm (per head) comes AFTER the rotation.  ``kout`` (k's shape): the prepared keys go there and
+    ``k`` stays as it is, so that ``v`` may be ``k`` itself.  The last
+    ``ring`` real tokens of each row go to ``kcache [slots, ring, GK, D]`` / ``vcache [slots, ring, G, V]`` at row
     ``position mod ring``.  ``k`` None (then ``v`` and the caches too): only the queries are prepared."""
     if _cuda(q):
         _ext.count_launch()
-        ext().window_qk_prepare(q, k, v, qw, kw, norm_all, eps, inv_freq, rot_dims if inv_freq is not None else 0, _i32(pos0), _i32(lens),
-                                _i32(slots), kcache, vcache)
+        ext().window_qk_prepare(q, k, v, kout, qw, kw, norm_all, unit, eps, inv_freq, rot_dims if inv_freq is not None else 0, float(amp),
+                                _i32(pos0), _i32(lens), _i32(slots), kcache, vcache)
         return
     B, S = q.shape[:2]
     pos = (pos0.long()[:, None] + torch.arange(S)[None, :])[:, :, None]
@@ -692,20 +719,23 @@ def window_qk_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[to
         elif w is not None:
             f = f / torch.sqrt(f.pow(2).mean(-1, keepdim=True) + eps) * w
         if inv_freq is not None and rot_dims:
-            f = _rotate(f, pos, inv_freq, rot_dims)
+            f = _rotate(f, pos, inv_freq, rot_dims, amp)
+        if unit:
+            f = f / torch.sqrt(f.pow(2).mean(-1, keepdim=True) + eps)
         return f.to(x.dtype)
 
-    if qw is not None or inv_freq is not None:
+    if qw is not None or inv_freq is not None or unit:
         q.copy_(prep(q, qw))
     if k is None:
         return
-    if kw is not None or inv_freq is not None:
-        k.copy_(prep(k, kw))
+    done = k if kout is None else kout
+    if kw is not None or inv_freq is not None or unit or kout is not None:
+        done.copy_(prep(k, kw))
     ring = kcache.shape[1]
     for b in range(B):
         n, p0, sl = int(lens[b]), int(pos0[b]), int(slots[b])
         for t in range(max(0, n - ring), n):
-            kcache[sl, (p0 + t) % ring] = k[b, t]
+            kcache[sl, (p0 + t) % ring] = done[b, t]
             vcache[sl, (p0 + t) % ring] = v[b, t]
 
 
@@ -713,66 +743,86 @@ def _capped(sc: torch.Tensor, softcap: float) -> torch.Tensor:
     return softcap * torch.tanh(sc / softcap) if softcap > 0 else sc
 
 
-def _window_weights(sc: torch.Tensor, ok: torch.Tensor, score_bias: Optional[torch.Tensor]) -> torch.Tensor:
-    """``sc [B,H,...,keys]`` scores, ``ok`` broadcastable → weights: a softmax over the visible keys, or with ``score_bias [H]``
-    ``sigmoid(score + bias[h])`` of every visible key by itself."""
-    if score_bias is None:
-        return torch.nan_to_num(torch.softmax(sc.masked_fill(~ok, float("-inf")), -1), nan=0.0)
-    bias = score_bias.view((1, -1) + (1,) * (sc.dim() - 2))
-    return torch.sigmoid(sc + bias) * ok
+def _window_heads(sc: torch.Tensor, v: torch.Tensor, ok: torch.Tensor, score_bias, sink, diff) -> torch.Tensor:
+    """Scores ``sc [B,H*maps,Q,K]``, ``v [B,K,G,V]``, ``ok`` broadcastable → the heads' results ``[B,Q,H,V]``.  Weights: a softmax over the
+    visible keys (with ``exp(sink[h])`` in the denominator), or with ``score_bias [H]`` ``sigmoid(score + bias[h])`` of every visible key by
+    itself; two maps are joined."""
+    w = _sink_softmax(sc, sink, ok) if score_bias is None else torch.sigmoid(sc + score_bias.view(1, -1, 1, 1)) * ok
+    o = torch.einsum("bhqk,bkhv->bqhv", w, v.repeat_interleave(w.shape[1] // v.shape[2], 2))
+    if diff is None:
+        return o
+    lam, eps, post = diff
+    o = o.unflatten(2, (-1, 2))
+    o = o[:, :, :, 0] - lam.float() * o[:, :, :, 1]
+    return o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * post
+
+
+def _map_keys(k: torch.Tensor, heads: int, maps: int) -> torch.Tensor:
+    """``k [B,K,G*maps,D]`` → the key of every query head and map ``[B,K,H*maps,D]``."""
+    g = k.unflatten(2, (-1, maps))
+    return g.repeat_interleave(heads // g.shape[2], 2).flatten(2, 3)
 
 
 def window_attention_prompt(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: Optional[torch.Tensor], lens: torch.Tensor,
                             window: int, scale: float, softcap: float, out: torch.Tensor, out_scale: float = 1.0,
-                            score_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                            score_bias: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0,
+                            diff=None) -> torch.Tensor:
     """Prompts that start at position 0: ``q [B,S,H,D]``, ``k [B,S,G,D]``, ``v [B,S,G,V]`` (views), query head h uses key/value head
-    ``h // (H/G)``; query i sees ``i - window < j <= i``.  Scores ``q.k * scale``, capped as ``softcap * tanh(score / softcap)``
-    when ``softcap > 0``, softmax in float; with ``score_bias [H]`` (float) the weight of a visible key is
-    ``sigmoid(score + score_bias[h])`` instead, not normalised over the keys.  Each head's result is multiplied by
+    ``h // (H/G)``; query i sees ``i - window < j <= i`` and, with ``chunk > 0``, only ``j // chunk == i // chunk``.  Scores ``q.k * scale``,
+    capped as ``softcap * tanh(score / softcap)``
+    when ``softcap > 0``, softmax in float, ``exp(sink[h])`` (``sink [H]`` float, optional) in its denominator; with ``score_bias [H]``
+    (float) the weight of a visible key is
+    ``sigmoid(score + score_bias[h])`` instead, not normalised over the keys.  ``diff = (lam [1] float, eps, post)``: two score maps per head,
+    ``q [B,S,2H,D]`` and ``k [B,S,2G,D]`` hold each head's (group's) two side by side, every map is a softmax over the same values, and a
+    head's result is ``unit(a1 - lam a2) * post`` with ``unit(o) = o / sqrt(mean(o^2) + eps)``.  Each head's result is multiplied by
     ``sigmoid(gate[b,s,h])`` (if given) and ``out_scale`` and written to ``out [B*S, >= H*V]`` (row stride free); padded rows give
     zeros."""
+    lam, eps, post = diff if diff is not None else (None, 0.0, 1.0)
     if _cuda(q):
         _ext.count_launch()
-        ext().window_attention_prompt(q, k, v, gate, _i32(lens), window, scale, softcap, score_bias, out, out_scale)
+        ext().window_attention_prompt(q, k, v, gate, _i32(lens), window, chunk, scale, softcap, score_bias, sink, lam, eps, post, out, out_scale)
         return out
-    B, S, H, D = q.shape
-    G, V = k.shape[2], v.shape[3]
-    kk, vv = k.float().repeat_interleave(H // G, 2), v.float().repeat_interleave(H // G, 2)
-    sc = _capped(torch.einsum("bihd,bjhd->bhij", q.float(), kk) * scale, softcap)
+    maps = 2 if diff is not None else 1
+    B, S, H, V = q.shape[0], q.shape[1], q.shape[2] // maps, v.shape[3]
+    sc = _capped(torch.einsum("bihd,bjhd->bhij", q.float(), _map_keys(k.float(), H, maps)) * scale, softcap)
     i, j = torch.arange(S)[:, None], torch.arange(S)[None, :]
     real = (torch.arange(S)[None, :] < lens[:, None])
-    vv = torch.where(real[..., None, None], vv, torch.zeros(()))
+    vv = torch.where(real[..., None, None], v.float(), torch.zeros(()))
     sc = torch.where(real[:, None, None, :], sc, torch.zeros(()))                               # padded rows hold anything
-    o = torch.einsum("bhij,bjhv->bihv", _window_weights(sc, ((j <= i) & (j > i - window))[None, None], score_bias), vv)
+    o = _window_heads(sc, vv, _visible(i, j, chunk, window)[None, None], score_bias, sink, diff)
     if gate is not None:
         o = o * torch.sigmoid(gate.float())[..., None]
-    o = torch.where((torch.arange(S)[None, :] < lens[:, None])[..., None, None], o * out_scale, torch.zeros_like(o))
+    o = torch.where(real[..., None, None], o * out_scale, torch.zeros_like(o))
     out[:, :H * V] = o.reshape(B * S, H * V).to(out.dtype)
     return out
 
 
 def window_attention_token(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, gate: Optional[torch.Tensor], slots: torch.Tensor,
                            pos0: torch.Tensor, lens: torch.Tensor, window: int, scale: float, softcap: float, out: torch.Tensor,
-                           out_scale: float = 1.0, score_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                           out_scale: float = 1.0, score_bias: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
+                           chunk: int = 0, diff=None) -> torch.Tensor:
     """Single tokens ``q [B,1,H,D]`` at positions ``pos0`` against their slots' rings (``kcache [slots, ring, G, D]``, ``vcache
-    [slots, ring, G, V]``; row ``j mod ring`` holds position j, the token's own row included; ``ring >= window``).  Same scores,
-    weights, gate and output layout as :func:`window_attention_prompt`; rows with ``lens == 0`` give zeros."""
+    [slots, ring, G, V]``; row ``j mod ring`` holds position j, the token's own row included; the ring is at least as long as the longest
+    visible stretch).  Same scores,
+    weights, maps (``kcache [slots, ring, 2G, D]``), gate and output layout as :func:`window_attention_prompt`; rows with ``lens == 0`` give
+    zeros."""
+    lam, eps, post = diff if diff is not None else (None, 0.0, 1.0)
     if _cuda(q):
         _ext.count_launch()
-        ext().window_attention_token(q, kcache, vcache, gate, _i32(slots), _i32(pos0), _i32(lens), window, scale, softcap, score_bias, out,
-                                     out_scale)
+        ext().window_attention_token(q, kcache, vcache, gate, _i32(slots), _i32(pos0), _i32(lens), window, chunk, scale, softcap, score_bias, sink,
+                                     lam, eps, post, out, out_scale)
         return out
-    B, _, H, D = q.shape
-    ring, G, V = kcache.shape[1], kcache.shape[2], vcache.shape[3]
-    kb = kcache[slots.long()].float().repeat_interleave(H // G, 2)                                  # [B, ring, H, D]
-    vb = vcache[slots.long()].float().repeat_interleave(H // G, 2)
+    maps = 2 if diff is not None else 1
+    B, H, V = q.shape[0], q.shape[2] // maps, vcache.shape[3]
+    ring = kcache.shape[1]
+    kb, vb = _map_keys(kcache[slots.long()].float(), H, maps), vcache[slots.long()].float()          # [B, ring, heads, D], [B, ring, G, V]
     sc = _capped(torch.einsum("bhd,brhd->bhr", q[:, 0].float(), kb) * scale, softcap)
     p = pos0.long()[:, None]
-    m = torch.remainder(p - torch.arange(ring)[None, :], ring)                                      # distance back of ring row r
-    ok = (p - m >= 0) & (m < window)
+    j = p - torch.remainder(p - torch.arange(ring)[None, :], ring)                                   # position held by ring row r
+    ok = _visible(p, j, chunk, window)
     sc = torch.where(ok[:, None, :], sc, torch.zeros(()))
     vb = torch.where(ok[:, :, None, None], vb, torch.zeros_like(vb))                               # rows never written hold anything
-    o = torch.einsum("bhr,brhv->bhv", _window_weights(sc, ok[:, None, :], score_bias), vb)
+    o = _window_heads(sc[:, :, None, :], vb, ok[:, None, None, :], score_bias, sink, diff)[:, 0]
     if gate is not None:
         o = o * torch.sigmoid(gate.float()).view(B, H, 1)
     o = torch.where((lens > 0)[:, None, None], o * out_scale, torch.zeros_like(o))
@@ -841,14 +891,15 @@ def ssd_scan(x: torch.Tensor, bm: torch.Tensor, cm: torch.Tensor, dtraw: torch.T
 
 
 # ------------------------------------------------------------------------------------------------ gated feed-forward, output gates
-def clamped_glu(gu: torch.Tensor, limit: float, slope: float) -> torch.Tensor:
-    """``gu [M, 2F]`` (gate columns, then up columns) → ``[M, F]``: ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``,
-    ``g * sigmoid(slope * g) * (u + 1)``."""
+def clamped_glu(gu: torch.Tensor, limit: float, slope: float, row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``gu [M, 2F]`` (gate columns, then up columns), times ``row_scale [M]`` (float, optional) → ``[M, F]``: ``g = min(gate, limit)``,
+    ``u = clamp(up, -limit, limit)``, ``g * sigmoid(slope * g) * (u + 1)``."""
     if _cuda(gu):
         _ext.count_launch()
-        return ext().clamped_glu(gu, float(limit), float(slope))
+        return ext().clamped_glu(gu, float(limit), float(slope), row_scale)
     half = gu.shape[1] // 2
-    g, u = gu[:, :half].float().clamp(max=limit), gu[:, half:].float().clamp(-limit, limit)
+    f = gu.float() if row_scale is None else gu.float() * row_scale.reshape(-1, 1)
+    g, u = f[:, :half].clamp(max=limit), f[:, half:].clamp(-limit, limit)
     return (g * torch.sigmoid(slope * g) * (u + 1.0)).to(gu.dtype)
 
 
