@@ -35,14 +35,16 @@ def parse():
     ap.add_argument("--steps", type=int, default=4)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--mode", default="train", choices=["train", "decode", "pp", "naguzen", "pinirax", "pulenex", "noresun", "kulisun"],
+    ap.add_argument("--mode", default="train", choices=["train", "decode", "pp", "naguzen", "pinirax", "pulenex", "noresun", "kulisun",
+                                                        "kekelix"],
                     help="train (default, the headline: Llama-2-7B training tokens/s) | decode (BASELINE config 5: Llama-2-13B "
                          "inference latency, batch 1, seq 2048) | pp (BASELINE config 4: GPT-NeoX-20B TP x PP=2 1F1B training) | "
                          "naguzen (serving throughput and per-kernel rooflines of the Naguzen design beside Llama at equal size) | "
                          "pinirax (the same for the Pinirax design beside Naguzen at equal size) | "
                          "pulenex (the same for the Pulenex design beside Naguzen and Pinirax at equal size) | "
                          "noresun (the same for the Noresun design beside Pinirax and Naguzen at equal size) | "
-                         "kulisun (the same for the Kulisun design beside Naguzen and Pulenex at equal size)")
+                         "kulisun (the same for the Kulisun design beside Naguzen and Pulenex at equal size) | "
+                         "kekelix (the same for the Kekelix design beside Noresun and Kulisun at equal size)")
     ap.add_argument("--seq", type=int, default=4096)
     ap.add_argument("--global-batch", type=int, default=4)
     ap.add_argument("--layers", type=int, default=32, help="32 = Llama-2-7B (anything else is a debug run)")
@@ -185,6 +187,10 @@ def main():
             import bench_kulisun
 
             return bench_kulisun.main(args)
+        if args.mode == "kekelix":
+            import bench_kekelix
+
+            return bench_kekelix.main(args)
         if args.mode == "pulenex":
             import bench_pulenex
 

@@ -280,8 +280,9 @@ bool route_topk(const float* logits, long z_stride, const float* correction, int
     return true;
 }
 
-// out[n, o] = w[o, :] . x[n, :] in float for a few rows n (a warp per output; w float or bfloat16, x float or bfloat16)
-template <typename Tw, typename Tx>
+// out[n, o] = w[o, :] . x[n, :] in float for a few rows n (a warp per output; w float or bfloat16, x float or bfloat16).  VEC: four
+// consecutive inputs per lane and access, four accesses in flight.
+template <typename Tw, typename Tx, bool VEC>
 __global__ void small_linear_f32_kernel(const Tw* __restrict__ w, const Tx* __restrict__ x, long x_stride, int N, int O, int I,
                                         float* __restrict__ out) {
     const int o = blockIdx.x * blockDim.y + threadIdx.y, n = blockIdx.y, lane = threadIdx.x;
@@ -289,18 +290,42 @@ __global__ void small_linear_f32_kernel(const Tw* __restrict__ w, const Tx* __re
     const Tw* wr = w + (long)o * I;
     const Tx* xr = x + (long)n * x_stride;
     float acc = 0.f;
-    for (int i = lane; i < I; i += 32) acc = fmaf(ldf(wr + i), ldf(xr + i), acc);
+    if (VEC) {
+        float part[4] = {0.f, 0.f, 0.f, 0.f};
+        int i = lane * 4;
+        for (; i + 384 < I; i += 512) {
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const float4 a = ld4(wr + i + 128 * u), b = ld4(xr + i + 128 * u);
+                part[u] = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, part[u]))));
+            }
+        }
+        for (; i < I; i += 128) {
+            const float4 a = ld4(wr + i), b = ld4(xr + i);
+            acc = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc))));
+        }
+        acc += (part[0] + part[1]) + (part[2] + part[3]);
+    } else {
+        for (int i = lane; i < I; i += 32) acc = fmaf(ldf(wr + i), ldf(xr + i), acc);
+    }
     acc = warp_sum(acc);
     if (lane == 0) out[(long)n * O + o] = acc;
 }
 
+template <typename Tw, typename Tx>
+static void small_linear_launch(const void* w, const void* x, long x_stride, int N, int O, int I, float* out, cudaStream_t s) {
+    dim3 block(32, 4), grid((O + 3) / 4, N);
+    const bool vec = I % 4 == 0 && x_stride % 4 == 0 && (uintptr_t)w % (4 * sizeof(Tw)) == 0 && (uintptr_t)x % (4 * sizeof(Tx)) == 0;
+    if (vec) small_linear_f32_kernel<Tw, Tx, true><<<grid, block, 0, s>>>((const Tw*)w, (const Tx*)x, x_stride, N, O, I, out);
+    else small_linear_f32_kernel<Tw, Tx, false><<<grid, block, 0, s>>>((const Tw*)w, (const Tx*)x, x_stride, N, O, I, out);
+}
+
 void small_linear_f32(const void* w, int w_bf, const void* x, int x_bf, long x_stride, int N, int O, int I, float* out, cudaStream_t s) {
     if (N * O == 0) return;
-    dim3 block(32, 8), grid((O + 7) / 8, N);
-    if (w_bf && x_bf) small_linear_f32_kernel<bf16, bf16><<<grid, block, 0, s>>>((const bf16*)w, (const bf16*)x, x_stride, N, O, I, out);
-    else if (!w_bf && x_bf) small_linear_f32_kernel<float, bf16><<<grid, block, 0, s>>>((const float*)w, (const bf16*)x, x_stride, N, O, I, out);
-    else if (w_bf && !x_bf) small_linear_f32_kernel<bf16, float><<<grid, block, 0, s>>>((const bf16*)w, (const float*)x, x_stride, N, O, I, out);
-    else small_linear_f32_kernel<float, float><<<grid, block, 0, s>>>((const float*)w, (const float*)x, x_stride, N, O, I, out);
+    if (w_bf && x_bf) small_linear_launch<bf16, bf16>(w, x, x_stride, N, O, I, out, s);
+    else if (!w_bf && x_bf) small_linear_launch<float, bf16>(w, x, x_stride, N, O, I, out, s);
+    else if (w_bf && !x_bf) small_linear_launch<bf16, float>(w, x, x_stride, N, O, I, out, s);
+    else small_linear_launch<float, float>(w, x, x_stride, N, O, I, out, s);
 }
 
 void xielu(const void* x, void* out, int bf, long n, float ap, float an, cudaStream_t s) {

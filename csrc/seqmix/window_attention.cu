@@ -113,6 +113,127 @@ __global__ void window_qk_prepare_kernel(T* q, long q_sb, long q_st, T* k, long 
     }
 }
 
+// The same for heads of at most 32 E coordinates (E = 4 or 8) whose rows start on whole fours and whose rotated halves are whole E: a warp
+// holds a head, E consecutive coordinates per lane, read once; a pair's other half comes from the lane half / E away.
+template <typename T, int E>
+__global__ void __launch_bounds__(256)
+window_qk_prepare_vec_kernel(T* q, long q_sb, long q_st, T* k, long k_sb, long k_st, T* kout, long ko_sb, long ko_st, const T* v, long v_sb,
+                             long v_st, const float* __restrict__ qw, const float* __restrict__ kw, int norm_all, int unit, float eps,
+                             const float* __restrict__ inv_freq, int dims, float amp, const int* __restrict__ pos0,
+                             const int* __restrict__ lens, const int* __restrict__ slots, T* kcache, T* vcache, int ring, int S, int H, int GK,
+                             int G, int D, int V) {
+    extern __shared__ __align__(16) float trig[];            // cos, then sin, of the token's angles (times amp)
+    __shared__ float red[2][8];
+    const int row = blockIdx.x, b = row / S, t = row - b * S, lane = threadIdx.x, tid = threadIdx.y * 32 + lane;
+    const int len = min(lens[b], S);
+    if (t >= len) return;
+    const bool keep = k != nullptr && t >= len - ring;
+    const int pos = pos0[b] + t, half = inv_freq ? dims / 2 : 0, rot = 2 * half;
+    const long cr = k ? (long)slots[b] * ring + pos % ring : 0;
+    T* qrow = q + (long)b * q_sb + (long)t * q_st;
+    T* krow = k ? k + (long)b * k_sb + (long)t * k_st : nullptr;
+    T* korow = k ? kout + (long)b * ko_sb + (long)t * ko_st : nullptr;
+    for (int i = tid; i < half; i += 256) {
+        float sn, cs;
+        sincosf((float)pos * inv_freq[i], &sn, &cs);
+        trig[i] = cs * amp; trig[half + i] = sn * amp;
+    }
+    if (norm_all) {
+        float sq = 0.f, sk = 0.f;
+        if (qw) for (int x = tid * 4; x < H * D; x += 1024) { const float4 e = ld4(qrow + x); sq += e.x * e.x + e.y * e.y + e.z * e.z + e.w * e.w; }
+        if (kw && krow) for (int x = tid * 4; x < GK * D; x += 1024) { const float4 e = ld4(krow + x); sk += e.x * e.x + e.y * e.y + e.z * e.z + e.w * e.w; }
+        sq = warp_sum(sq); sk = warp_sum(sk);
+        if (lane == 0) { red[0][threadIdx.y] = sq; red[1][threadIdx.y] = sk; }
+    }
+    if (norm_all || half) __syncthreads();
+    float inv_all[2] = {1.f, 1.f};
+    if (norm_all) {
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int x = 0; x < 8; ++x) { sq += red[0][x]; sk += red[1][x]; }
+        inv_all[0] = 1.f / sqrtf(sq / (float)(H * D) + eps);
+        inv_all[1] = 1.f / sqrtf(sk / (float)(GK * D) + eps);
+    }
+    auto load = [](float (&x)[E], const T* src) {
+#pragma unroll
+        for (int e = 0; e < E; e += 4) { const float4 a = ld4(src + e); x[e] = a.x; x[e + 1] = a.y; x[e + 2] = a.z; x[e + 3] = a.w; }
+    };
+    auto loadf = [](float (&x)[E], const float* src) {
+#pragma unroll
+        for (int e = 0; e < E; e += 4) { const float4 a = ld4(src + e); x[e] = a.x; x[e + 1] = a.y; x[e + 2] = a.z; x[e + 3] = a.w; }
+    };
+    auto store = [](T* dst, const float (&x)[E]) {
+#pragma unroll
+        for (int e = 0; e < E; e += 4) st4(dst + e, make_float4(x[e], x[e + 1], x[e + 2], x[e + 3]));
+    };
+    const int c = lane * E, shift = half / E;                // this lane's coordinates; lanes between the members of a pair
+    const bool in = c < D;
+    const bool touch_q = qw || rot || unit;                  // otherwise the queries stay as they are
+    const int first = touch_q ? 0 : H, units = krow ? H + GK + (keep ? G : 0) : H;
+    for (int u = first + threadIdx.y; u < units; u += 8) {
+        if (u < H + GK) {
+            const bool isq = u < H;
+            const int hh = isq ? u : u - H;
+            const T* p = (isq ? qrow : krow) + (long)hh * D;
+            T* o = (isq ? qrow : korow) + (long)hh * D;
+            const float* w = isq ? qw : kw;
+            float x[E];
+            if (in) load(x, p + c);
+            else {
+#pragma unroll
+                for (int e = 0; e < E; ++e) x[e] = 0.f;
+            }
+            float inv = 1.f;
+            if (w && norm_all) {
+                inv = inv_all[isq ? 0 : 1];
+                w += (long)hh * D;
+            } else if (w || unit) {
+                const float a = unit && c < rot ? amp : 1.f;
+                float ss = 0.f;
+#pragma unroll
+                for (int e = 0; e < E; ++e) ss = fmaf(x[e] * a, x[e] * a, ss);
+                inv = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
+            }
+            if (w && in) {
+                float g[E];
+                loadf(g, w + c);
+#pragma unroll
+                for (int e = 0; e < E; ++e) x[e] *= inv * g[e];
+            }
+            if (rot) {
+                const bool low = c < half, turn = c < rot;
+                const int other = turn ? (low ? lane + shift : lane - shift) : lane;
+                float y[E];
+#pragma unroll
+                for (int e = 0; e < E; ++e) y[e] = __shfl_sync(0xffffffffu, x[e], other);
+                if (turn) {
+                    const float* cs = trig + (low ? c : c - half);
+#pragma unroll
+                    for (int e = 0; e < E; ++e) {
+                        const float sn = cs[half + e];
+                        x[e] = low ? x[e] * cs[e] - y[e] * sn : x[e] * cs[e] + y[e] * sn;
+                    }
+                }
+            }
+            if (unit) {
+#pragma unroll
+                for (int e = 0; e < E; ++e) x[e] *= inv;
+            }
+            if (!in) continue;
+            if (w || rot || unit || o != p) store(o + c, x);
+            if (!isq && keep) store(kcache + (cr * GK + hh) * D + c, x);
+        } else {
+            const int hh = u - H - GK;
+            const T* p = v + (long)b * v_sb + (long)t * v_st + (long)hh * V;
+            T* dst = vcache + (cr * G + hh) * V;
+            for (int d = lane * 4; d < V; d += 128) {
+                if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst + d) = *reinterpret_cast<const uint2*>(p + d);
+                else *reinterpret_cast<uint4*>(dst + d) = *reinterpret_cast<const uint4*>(p + d);
+            }
+        }
+    }
+}
+
 __device__ __forceinline__ float cap_score(float s, float softcap, float inv_cap) { return softcap > 0.f ? softcap * tanhf(s * inv_cap) : s; }
 
 constexpr int kKeys = 32;       // keys per shared-memory chunk
@@ -383,19 +504,19 @@ __global__ void __launch_bounds__(128) window_token_kernel(
 
 // grid (H, B), 8 warps: the stretches' partial softmaxes of one (sequence, head) folded, with the sink in the denominator; the maps joined;
 // gated, scaled and written.  A warp adds every eighth stretch; the warps' sums meet in shared memory.
-// shared: weights [maps][splits], sums [8][V], heads [maps][V], one float per warp
+// shared: sums [8][V], heads [maps][V], one float per warp, weights [maps][splits]
 template <typename T>
 __global__ void __launch_bounds__(256) window_token_merge_kernel(const float* __restrict__ part_m, const float* __restrict__ part_l,
                                                                  const float* __restrict__ part_acc, const T* __restrict__ gate, long g_sb,
                                                                  int H, int V, int splits, const int* __restrict__ lens,
                                                                  const WindowRule rule, T* __restrict__ out, long out_stride,
                                                                  float out_scale) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     const int M = rule.maps, h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    float* Ws = sm;
-    float* Rs = Ws + M * splits;
+    float* Rs = sm;
     float* As = Rs + 8 * V;
     float* red = As + M * V;
+    float* Ws = red + 8;
     T* dst = out + (long)b * out_stride + (long)h * V;
     if (lens[b] <= 0) {
         for (int c = tid; c < V; c += 256) stf(dst + c, 0.f);
@@ -410,22 +531,36 @@ __global__ void __launch_bounds__(256) window_token_merge_kernel(const float* __
         for (int w = 16; w > 0; w >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, w));
         float lt = 0.f;
         for (int s = lane; s < splits; s += 32) {
-            const float pm = part_m[o + s], e = pm > -INFINITY ? expf(pm - mt) : 0.f;
+            const float pm = part_m[o + s], pl = part_l[o + s], e = pm > -INFINITY ? expf(pm - mt) : 0.f;
             if (warp == 0) Ws[a * splits + s] = e;
-            if (e > 0.f) lt = fmaf(part_l[o + s], e, lt);
+            lt = fmaf(pl, e, lt);
         }
         lt = warp_sum(lt);
         if (rule.sink) lt += expf(rule.sink[hh] - mt);
         const float inv = lt > 0.f ? 1.f / lt : 0.f;
         __syncthreads();
-        for (int c = lane; c < V; c += 32) {
-            float acc = 0.f;
+        if (V % 4 == 0) {                                            // a stretch that saw nothing left its sums unwritten: not added
+            for (int c = lane * 4; c < V; c += 128) {
+                float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
-            for (int s = warp; s < splits; s += 8) {
-                const float e = Ws[a * splits + s];
-                if (e > 0.f) acc = fmaf(part_acc[(o + s) * V + c], e, acc);
+                for (int s = warp; s < splits; s += 8) {
+                    const float e = Ws[a * splits + s];
+                    const float4 x = ld4(part_acc + (o + s) * V + c);
+                    acc.x = e > 0.f ? fmaf(x.x, e, acc.x) : acc.x; acc.y = e > 0.f ? fmaf(x.y, e, acc.y) : acc.y;
+                    acc.z = e > 0.f ? fmaf(x.z, e, acc.z) : acc.z; acc.w = e > 0.f ? fmaf(x.w, e, acc.w) : acc.w;
+                }
+                st4(Rs + warp * V + c, acc);
             }
-            Rs[warp * V + c] = acc;
+        } else {
+            for (int c = lane; c < V; c += 32) {
+                float acc = 0.f;
+#pragma unroll 4
+                for (int s = warp; s < splits; s += 8) {
+                    const float e = Ws[a * splits + s], x = part_acc[(o + s) * V + c];
+                    acc = e > 0.f ? fmaf(x, e, acc) : acc;
+                }
+                Rs[warp * V + c] = acc;
+            }
         }
         __syncthreads();
         for (int c = tid; c < V; c += 256) {
@@ -463,13 +598,24 @@ void window_qk_prepare(void* q, long q_sb, long q_st, void* k, long k_sb, long k
                        void* vcache, int ring, int B, int S, int H, int GK, int G, int D, int V, cudaStream_t s) {
     if (B * S == 0) return;
     dim3 grid(B * S), block(32, 8);
-    const size_t smem = inv_freq ? sizeof(float) * dims : 0;
+    const size_t smem = inv_freq ? sizeof(float) * dims : 0, a4 = bf ? 8 : 16;
+    auto al = [&](const void* p, size_t n) { return p == nullptr || (uintptr_t)p % n == 0; };
+    const int half = inv_freq ? dims / 2 : 0, E = D <= 128 && half % 4 == 0 ? 4 : 8;
+    const bool vec = D % E == 0 && D <= 32 * E && half % E == 0 && (!k || V % 4 == 0) && al(q, a4) && al(k, a4) && al(kout, a4) && al(v, a4) &&
+                     al(kcache, a4) && al(vcache, a4) && al(qw, 16) && al(kw, 16) && q_sb % 4 == 0 && q_st % 4 == 0 && k_sb % 4 == 0 &&
+                     k_st % 4 == 0 && ko_sb % 4 == 0 && ko_st % 4 == 0 && v_sb % 4 == 0 && v_st % 4 == 0;
+#define SEQMIX_WQP_ARGS(T)                                                                                                            \
+    (T*)q, q_sb, q_st, (T*)k, k_sb, k_st, (T*)kout, ko_sb, ko_st, (const T*)v, v_sb, v_st, qw, kw, norm_all, unit, eps, inv_freq, dims,   \
+        amp, pos0, lens, slots, (T*)kcache, (T*)vcache, ring, S, H, GK, G, D, V
 #define SEQMIX_WQP(T)                                                                                                                 \
-    window_qk_prepare_kernel<T><<<grid, block, smem, s>>>((T*)q, q_sb, q_st, (T*)k, k_sb, k_st, (T*)kout, ko_sb, ko_st, (const T*)v, v_sb, \
-                                                          v_st, qw, kw, norm_all, unit, eps, inv_freq, dims, amp, pos0, lens, slots,     \
-                                                          (T*)kcache, (T*)vcache, ring, S, H, GK, G, D, V)
+    do {                                                                                                                              \
+        if (vec && E == 4) window_qk_prepare_vec_kernel<T, 4><<<grid, block, smem, s>>>(SEQMIX_WQP_ARGS(T));                            \
+        else if (vec) window_qk_prepare_vec_kernel<T, 8><<<grid, block, smem, s>>>(SEQMIX_WQP_ARGS(T));                                \
+        else window_qk_prepare_kernel<T><<<grid, block, smem, s>>>(SEQMIX_WQP_ARGS(T));                                                \
+    } while (0)
     if (bf) SEQMIX_WQP(bf16); else SEQMIX_WQP(float);
 #undef SEQMIX_WQP
+#undef SEQMIX_WQP_ARGS
 }
 
 static int value_cols_per_lane(int V) { return V <= 64 ? 2 : (V <= 128 ? 4 : (V <= 256 ? 8 : (V <= 512 ? 16 : 0))); }
