@@ -61,14 +61,14 @@ window_decode_mma_kernel(const bf16* __restrict__ q, long q_sb, const bf16* __re
     }
     const bf16* kb = kcache + ((long)slots[b] * ring * G + gr) * KD;
     const bf16* vb = vcache + ((long)slots[b] * ring * G + gr) * V;
-    const int kp8 = KD / 8, row8 = kp8 + V / 8;
+    const int kp8 = KD / 8, row8 = kp8 + V / 8, n = j1 - j0, first = j0 % ring;    // a stretch wraps at most once
     auto fetch = [&](int t) {                                                      // 16-byte pieces of 64 key and value rows
         bf16* Kd = St + (long)(t % stages) * kRows * (ldk + ldv);
         bf16* Vd = Kd + kRows * ldk;
         for (int r = warp; r < kRows; r += 8) {
-            const int j = j0 + t * kRows + r;
-            const bool on = j < j1;
-            const long row = (long)((on ? j : j1 - 1) % ring) * G;
+            const int i = t * kRows + r, at = first + min(i, n - 1);
+            const bool on = i < n;
+            const long row = (long)(at < ring ? at : at - ring) * G;
             for (int c = lane; c < row8; c += 32) {
                 if (c < kp8) cp16(Kd + r * ldk + c * 8, kb + row * KD + c * 8, on);
                 else cp16(Vd + r * ldv + (c - kp8) * 8, vb + row * V + (c - kp8) * 8, on);

@@ -32,9 +32,10 @@ window_prompt_mma_kernel(const bf16* __restrict__ q, long q_sb, long q_st, const
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int dk16 = DK / 16, vd16 = VD / 16, ldk = DK + kPad, ldv = VD + kPad;
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);          // [MAPS][kQT][ldk] queries, then key stage 1 (same size)
+    // the blocks of the last queries, which see the most keys, start first
     auto Kst = [&](int st) { return st ? Qs : Qs + MAPS * kQT * ldk; };                        // [MAPS][kKT][ldk] each
     auto Vst = [&](int st) { return Qs + MAPS * (kQT + kKT) * ldk + (st ? kKT * ldv : 0); };   // [kKT][ldv] each
-    const int q0 = blockIdx.x * kQT, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int q0 = (gridDim.z - 1 - blockIdx.z) * kQT, h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int hk = h / (H / G), map = warp >> 2;           // this warp's score map
     const int len = min(lens[b], S);
     bf16* ob = out + ((long)b * S) * out_stride + (long)h * VD;
@@ -259,7 +260,7 @@ static void prompt_launch(const bf16* q, long q_sb, long q_st, const bf16* k, lo
                           const bf16* gate, long g_sb, long g_st, const int* lens, int B, int S, int H, int G, int D, int V,
                           const WindowRule& rule, bf16* out, long out_stride, float out_scale, cudaStream_t s) {
     cudaFuncSetAttribute(window_prompt_mma_kernel<DK16, VD16, SIG, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-    window_prompt_mma_kernel<DK16, VD16, SIG, MAPS><<<dim3((S + kQT - 1) / kQT, H, B), 128 * MAPS, prompt_smem(D, V, MAPS), s>>>(
+    window_prompt_mma_kernel<DK16, VD16, SIG, MAPS><<<dim3(H, B, (S + kQT - 1) / kQT), 128 * MAPS, prompt_smem(D, V, MAPS), s>>>(
         q, q_sb, q_st, k, k_sb, k_st, v, v_sb, v_st, gate, g_sb, g_st, lens, S, H, G, D, V, rule, out, out_stride, out_scale);
 }
 
